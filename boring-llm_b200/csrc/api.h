@@ -66,7 +66,7 @@ int bl_gemm_skinny(const void* x, const void* w, const void* bias, int bias_dtyp
                    int M, int N, int K, int epilogue, void* stream);
 int bl_gemm_skinny_norm_parts(int N);
 int bl_gemm_skinny_residual_norm(const void* x, const void* w, void* out, int M, int N, int K, const void* norm_w,
-                                 int norm_w_dtype, void* hw, float* ss, void* stream);
+                                 int norm_w_dtype, void* hw, float* ss, const void* bias, int bias_dtype, void* stream);
 int bl_gemm_skinny_scaled(const void* hw, const void* w, const void* bias, int bias_dtype, void* out, int out_dtype,
                           int M, int N, int K, int epilogue, const float* ss, int parts, float eps, void* stream);
 
@@ -134,7 +134,7 @@ int bl_gemm_tc_pair_qkv_rope(const void* x, const void* w, const void* bias, int
 // the products that read the normed rows take hw and scale their accumulator rows by the row's 1 / sqrt(mean + eps).
 int bl_gemm_tc_pair_norm_parts(int M, int N);
 int bl_gemm_tc_pair_residual_norm(const void* x, const void* w, void* out, int M, int N, int K, const void* norm_w,
-                                  int norm_w_dtype, void* hw, float* ss, void* stream);
+                                  int norm_w_dtype, void* hw, float* ss, const void* bias, int bias_dtype, void* stream);
 int bl_gemm_tc_pair_swiglu_scaled(const void* hw, const void* w, void* out, int M, int N, int K, const float* ss,
                                   int parts, float inv_dim, float eps, void* stream);
 
@@ -377,6 +377,8 @@ int bl_gemm_plain_decay_exp(const float* x, int ldx, int x_tanh, const void* w, 
 int bl_post_norm_residual(float* x, const float* a, const void* wa, int wa_dtype, const float* b, const void* wb, int wb_dtype,
                           float rms_eps, const void* w, int w_dtype, float eps, void* y, int y_dtype, int rows, int d, void* stream);
 int bl_cast_rows(const float* x, void* y, int y_dtype, long long count, void* stream);
+// y[t] = [a[t] | b[t]] in y_dtype, rows of m and n 32-bit values.
+int bl_concat_rows(const float* a, int m, const float* b, int n, void* y, int y_dtype, int rows, void* stream);
 // out = (a / rms(a) * wa + b / rms(b) * wb) / 2 row by row (32-bit): the mean of two sublayer results, each RMS-normed first.
 int bl_pair_rms_mean(const float* a, const void* wa, int wa_dtype, const float* b, const void* wb, int wb_dtype, float rms_eps,
                      float* out, int rows, int d, void* stream);
@@ -419,11 +421,13 @@ int bl_moe_route(const float* z, int ldz, const void* correction, int corr_dtype
 int bl_expert_gemm_plain(const void* x, int x_dtype, int x_div, const void* w, int w_dtype, long long expert_stride, const int* ids,
                          void* out, int out_dtype, int P, int N, int K, int epilogue, const float* act, void* stream);
 int bl_moe_combine(const float* y, const float* wts, float* out, int T, int top, int d, int add, void* stream);
-// The same with further choices. bl_moe_route_ext: score_kind BL_SCORE_SIGMOID, or BL_SCORE_SOFTMAX (softmax of z over all E);
+// The same with further choices. bl_moe_route_ext: score_kind BL_SCORE_SIGMOID, or BL_SCORE_SOFTMAX (softmax of z over all E),
+// or BL_SCORE_CHOSEN (the choice runs on the logits themselves, the weights are the softmax over the chosen logits alone);
 // group_top 2: a group's score is the sum of its two largest choice scores, 1: its largest. Identity experts are the expert
 // numbers from n_real on: no matrix, no row in a product; the weighted sums take the token's input row x[t, :] for them.
 #define BL_SCORE_SIGMOID 0
 #define BL_SCORE_SOFTMAX 1
+#define BL_SCORE_CHOSEN 2
 int bl_moe_route_ext(const float* z, int ldz, const void* correction, int corr_dtype, int T, int E, int top, int n_groups, int keep,
                      int* ids, float* wts, int score_kind, int group_top, void* stream);
 int bl_expert_gemm_plain_some(const void* x, int x_dtype, int x_div, const void* w, int w_dtype, long long expert_stride,
@@ -458,8 +462,8 @@ int bl_glu_act(const float* x, long long ld_x, void* y, int y_dtype, long long l
 // cq = RMS norm of columns [off_q, off_q + q_rank) times q_norm_w (cq null: skipped), and into the token's page the row
 // [RMS norm of columns [off_kv, off_kv + rank) times kv_norm_w | the next rot_dim columns, the first 2 * rot_half of them
 // rotated in pairs (j, j + rot_half) by float(position) * inv_freq[j], cos and sin times mscale] (cache null: skipped);
-// cache [pages, page_size, rank + rot_dim]. bl_head_gemm_plain: out[t, h, n] = sum_k x[t, h, k] W[h][n, k] (* sigmoid(gate[t, h * N + n])),
-// every operand by its strides in elements. bl_rope_heads: out[t, h, out_off + .] = q[t, h, off + .] (n values, the
+// cache [pages, page_size, rank + rot_dim]. bl_head_gemm_plain: out[t, h, n] = sum_k x[t, h, k] W[h][n, k] (* sigmoid(gate[t, h * N + n]),
+// or with gate_heads sigmoid(gate[t, h])), every operand by its strides in elements. bl_rope_heads: out[t, h, out_off + .] = q[t, h, off + .] (n values, the
 // first 2 * rot_half rotated); with n_lead > 0 also lead_out[t, h, .] = lead[t, h, .] (n_lead values of every head, `lead` strided as q,
 // lead_out of out's dtype with strides of its own).
 // bl_latent_attention_plain: q [T, H, dk], out [T, H, dv]: softmax over the visible cached rows (window 0: all) of
@@ -470,7 +474,7 @@ int bl_latent_prep(const float* proj, int ld, int off_q, int q_rank, int off_kv,
                    int dtype, int T, void* stream);
 int bl_head_gemm_plain(const void* x, int x_dtype, long long ldx, long long x_head, const void* w, int w_dtype, long long w_head,
                        long long w_n, long long w_k, void* out, int out_dtype, long long ld_out, long long out_head, int T, int H,
-                       int N, int K, const float* gate, long long ld_gate, void* stream);
+                       int N, int K, const float* gate, long long ld_gate, int gate_heads, void* stream);
 int bl_rope_heads(const float* q, long long ld, long long head_stride, int off, const int* positions, const float* inv_freq,
                   int n, int rot_half, float mscale, void* out, int out_dtype, long long ld_out, long long out_head, int out_off, int T,
                   int H, const float* lead, int n_lead, void* lead_out, long long ld_lead, long long lead_head, void* stream);
@@ -490,7 +494,30 @@ int bl_latent_attention_mma(const void* q_lat, const void* q_rot, const void* ca
 // tile[i] = i / per for n_heads * per tiles; out[t, h * N + n] = hv[h, t, n] (* sigmoid(gate[t, h * N + n])) with hv [H, Tp, N] (latent.cu).
 int bl_head_tiles(int* tile, int n_heads, int per, void* stream);
 int bl_heads_gate_rows(const float* hv, const float* gate, long long ld_gate, void* out, int out_dtype, int T, int H, int N, int Tp,
-                       void* stream);
+                       int gate_heads, void* stream);
+
+// Attention whose heads' scores are mixed before the softmax (attention_mixed.cu): keys of unit root mean square, values =
+// keys times that root mean square. bl_mixed_prep: from a token's 32-bit projection (q from column 0, k from off_k): the
+// mixed queries q_out[t, h, c, :] = sum over the query heads g of key/value head c of talk[h, g] * normed q_g, the normed
+// keys into k_cache [pages, KV, page_size, dh], their root mean squares into k_rms [pages, KV, page_size] (entries
+// rms_stride floats apart). The attention kernels: score = q . (keys of all KV heads) * scale - slopes[h] (i - j) (slopes
+// null: none), softmax over j <= i, values of head h / (H / KV), optionally times sigmoid(gate[t, h * dh + d]); out
+// [T, H * dh]. _prefill walks 64-token tiles, _decode single-token requests (up to 16 slices of their keys, one cluster).
+int bl_mixed_prep(const float* proj, int ld, int off_k, const float* talk, float eps, const int* positions, const int* tok_req,
+                  const int* block_table, int max_pages, void* q_out, void* k_cache, float* k_rms, int rms_stride, int dtype, int T, int H,
+                  int KV, int dh, int page_size, void* stream);
+int bl_attention_mixed_plain(const void* q, const void* k_cache, const float* k_rms, int rms_stride, int dtype, const int* tok_req,
+                             const int* cu_q, const int* ctx_len, const int* block_table, int max_pages, const float* slopes,
+                             const float* gate, int ld_gate, void* out, int T, int H, int KV, int dh, int page_size, float scale,
+                             void* stream);
+int bl_attention_mixed_supported(int KV, int dh, int page_size);
+int bl_attention_mixed_decode_resident_blocks(int KV, int dh);
+int bl_attention_mixed_prefill(const void* q, const void* k_cache, const float* k_rms, const int* cu_q, const int* ctx_len,
+                               const int* block_table, int max_pages, const int* tiles, int n_tiles, void* out, int H, int KV, int dh,
+                               int page_size, float scale, const float* slopes, const float* gate, int ld_gate, void* stream);
+int bl_attention_mixed_decode(const void* q, const void* k_cache, const float* k_rms, const int* cu_q, const int* ctx_len,
+                              const int* block_table, int max_pages, const int* reqs, int n, int n_splits, void* out, int H, int KV, int dh,
+                              int page_size, float scale, const float* slopes, const float* gate, int ld_gate, void* stream);
 
 #ifdef __cplusplus
 }

@@ -13,7 +13,7 @@
 // Epilogues of the matrix products.
 #define BL_EPI_NONE 0      // out = acc
 #define BL_EPI_BIAS 1      // out = acc + bias[n]
-#define BL_EPI_RESIDUAL 2  // out (32-bit, in place) = out + acc
+#define BL_EPI_RESIDUAL 2  // out (32-bit, in place) = out + acc (+ bias[n], if a bias is given)
 #define BL_EPI_SWIGLU 3    // out[m, n] = silu(acc_gate[m, n]) * acc_up[m, n]; W holds gate rows then up rows
 #define BL_EPI_DECAY 4     // plain kernel only: out = exp(-coef[n / group] * softplus(sign * (acc + bias[n])))
 #define BL_EPI_DECAY_EXP 5 // plain kernel only: out = exp(-exp(acc + bias[n])), optionally with tanh on x as it is read
@@ -75,7 +75,9 @@ __device__ __forceinline__ float bl_glu(int kind, float g, float u, float limit)
     return bl_silu(g) * u;
 }
 // The gated epilogue of a product (BL_EPI_SWIGLU) computes silu(gate) * up unless the product's `bias` argument, which
-// that epilogue does not use otherwise, points to two 32-bit numbers {kind, limit}: then bl_glu(kind, gate, up, limit).
+// that epilogue does not use otherwise, points to 32-bit numbers {kind, limit}: then bl_glu(kind, gate, up, limit). With
+// kind + BL_GLU_BIASED the first four numbers {kind, limit, 0, 0} are followed by the biases that the sums get before the
+// activation, those of the N gate columns and then those of the N up columns.
 // bl_glu_fast: the same with the fast exponential and division of bl_silu_fast, for epilogues that round to bfloat16
 // (0.5 g (1 + tanh(z)) = g / (1 + e^(-2z)), so each form is one exponential and one division).
 __device__ __forceinline__ float bl_glu_fast(int kind, float g, float u, float limit) {
@@ -88,13 +90,15 @@ __device__ __forceinline__ float bl_glu_fast(int kind, float g, float u, float l
     }
     return __fdividef(g, 1.0f + __expf(-g)) * u;
 }
-struct BlGluArgs { int kind; float limit; };
-__device__ __forceinline__ BlGluArgs bl_glu_args(const void* two_numbers) {
-    BlGluArgs a{BL_GLU_SILU, 0.f};
-    if (two_numbers != nullptr) {
-        const float* f = reinterpret_cast<const float*>(two_numbers);
+#define BL_GLU_BIASED 16
+struct BlGluArgs { int kind; float limit; const float* bias; };
+__device__ __forceinline__ BlGluArgs bl_glu_args(const void* numbers) {
+    BlGluArgs a{BL_GLU_SILU, 0.f, nullptr};
+    if (numbers != nullptr) {
+        const float* f = reinterpret_cast<const float*>(numbers);
         a.kind = (int)f[0];
         a.limit = f[1];
+        if (a.kind >= BL_GLU_BIASED) { a.kind -= BL_GLU_BIASED; a.bias = f + 4; }
     }
     return a;
 }

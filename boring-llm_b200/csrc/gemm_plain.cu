@@ -72,8 +72,15 @@ gemm_plain_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const void
             TO* dst = out + (size_t)m * N + n;
             float v = acc[i][j];
             if (EPI == BL_EPI_BIAS) v += bl_load_any(bias, bias_dtype, n);
-            if (EPI == BL_EPI_RESIDUAL) v += bl_load(dst);
-            if (EPI == BL_EPI_SWIGLU) v = bl_glu(glu.kind, v, acu[i][j], glu.limit);
+            if (EPI == BL_EPI_RESIDUAL) {
+                if (bias) v += bl_load_any(bias, bias_dtype, n);
+                v += bl_load(dst);
+            }
+            if (EPI == BL_EPI_SWIGLU) {
+                float u = acu[i][j];
+                if (glu.bias) { v += glu.bias[n]; u += glu.bias[N + n]; }
+                v = bl_glu(glu.kind, v, u, glu.limit);
+            }
             if (EPI == BL_EPI_DECAY) {                 // exp(-coef[head] * softplus(sign * (acc + bias))), head = n / group
                 if (bias) v += bl_load_any(bias, bias_dtype, n);
                 const float u = sign * v;

@@ -139,12 +139,12 @@ gemm_skinny_kernel(const __nv_bfloat16* x /* written by the kernel before: no re
     const int e_n = n0 + e_c, e_m = m0 + e_tok;
     const bool e_ok = threadIdx.x < COLS * TOK && e_n < N && e_m < M && part == 0;
     float e_add = 0.f;
-    if (EPI == BL_EPI_BIAS && e_ok) e_add = bl_load_any(bias, bias_dtype, e_n);
+    if ((EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) && e_ok) e_add = bl_load_any(bias, bias_dtype, e_n);
     const bool begins_norm = EPI == BL_EPI_RESIDUAL && lk.hw != nullptr;
     float e_nw = 0.f;                                             // the next norm's weight of this thread's column
     if (begins_norm && e_ok) e_nw = bl_load_any(lk.norm_w, lk.norm_w_dtype, e_n);
     bl_pdl_wait();
-    if (EPI == BL_EPI_RESIDUAL && e_ok) e_add = bl_load(out + (size_t)e_m * N + e_n);   // on its way during the product
+    if (EPI == BL_EPI_RESIDUAL && e_ok) e_add += bl_load(out + (size_t)e_m * N + e_n);  // on its way during the product
     fetch_x(b0, k_begin + warp * 32);
     if (lk.ss_in != nullptr) {
         // the scale of each of this block's rows, while the product's operands are on their way: warp w adds up the
@@ -216,8 +216,18 @@ gemm_skinny_kernel(const __nv_bfloat16* x /* written by the kernel before: no re
             if (SPLIT == 2) v += peer_sums[i];
             if (lk.ss_in != nullptr) { const float r = row_scale[tok]; v *= r; if (GLU) u *= r; }
             TO* dst = out + (size_t)m * N + n;
-            if (EPI == BL_EPI_BIAS || EPI == BL_EPI_RESIDUAL) v += (i == threadIdx.x) ? e_add : (EPI == BL_EPI_BIAS ? bl_load_any(bias, bias_dtype, n) : bl_load(dst));
-            if (GLU) v = bl_glu(glu.kind, v, u, glu.limit);
+            if (EPI == BL_EPI_BIAS || EPI == BL_EPI_RESIDUAL) {
+                float add = e_add;
+                if (i != threadIdx.x) {
+                    add = EPI == BL_EPI_BIAS || bias != nullptr ? bl_load_any(bias, bias_dtype, n) : 0.f;
+                    if (EPI == BL_EPI_RESIDUAL) add += bl_load(dst);
+                }
+                v += add;
+            }
+            if (GLU) {
+                if (glu.bias) { v += glu.bias[n]; u += glu.bias[N + n]; }
+                v = bl_glu(glu.kind, v, u, glu.limit);
+            }
             bl_store(dst, v);
         }
         if (begins_norm) {                                        // (the same for the whole block)
@@ -318,7 +328,10 @@ gemm_skinny_cols_kernel(const __nv_bfloat16* x /* written by the kernel before: 
             TO* dst = out + (size_t)m * N + (hi ? r_hi : r_lo);
             float v = acc[j][i];
             if (EPI == BL_EPI_BIAS) v += hi ? e_hi : e_lo;
-            if (EPI == BL_EPI_RESIDUAL) v += bl_load(dst);
+            if (EPI == BL_EPI_RESIDUAL) {
+                if (bias != nullptr) v += bl_load_any(bias, bias_dtype, hi ? r_hi : r_lo);
+                v += bl_load(dst);
+            }
             bl_store(dst, v);
         }
     }
@@ -445,16 +458,17 @@ extern "C" int bl_gemm_skinny(const void* x, const void* w, const void* bias, in
 // Partial sums of squares per row that the linked residual product writes: one per block of 16 columns.
 extern "C" int bl_gemm_skinny_norm_parts(int N) { return (N + COLS - 1) / COLS; }
 
-// out += x . W^T (32-bit residual stream, in place) and, for the RMS norm with weight norm_w that reads out next:
+// out += x . W^T (+ bias, if given; 32-bit residual stream, in place) and, for the RMS norm with weight norm_w that reads out next:
 // hw[M, N] = bfloat16(out * norm_w), ss[M, parts] = sums of squares of the new rows by block of 16 columns
 // (parts = bl_gemm_skinny_norm_parts(N)).
 extern "C" int bl_gemm_skinny_residual_norm(const void* x, const void* w, void* out, int M, int N, int K,
-                                            const void* norm_w, int norm_w_dtype, void* hw, float* ss, void* stream) {
+                                            const void* norm_w, int norm_w_dtype, void* hw, float* ss, const void* bias,
+                                            int bias_dtype, void* stream) {
     if (norm_w == nullptr || hw == nullptr || ss == nullptr || (norm_w_dtype != BL_F32 && norm_w_dtype != BL_BF16))
         BL_FAIL("bl_gemm_skinny_residual_norm: needs a float32 or bfloat16 norm weight, hw and ss");
     SkinnyLink lk = {};
     lk.norm_w = norm_w; lk.norm_w_dtype = norm_w_dtype; lk.hw = (__nv_bfloat16*)hw; lk.ss_out = ss;
-    return run(x, w, nullptr, 0, out, BL_F32, M, N, K, BL_EPI_RESIDUAL, lk, stream);
+    return run(x, w, bias, bias_dtype, out, BL_F32, M, N, K, BL_EPI_RESIDUAL, lk, stream);
 }
 
 // out = epilogue(r * (hw . W^T)) with r[m] = 1 / sqrt(sum(ss[m][:]) / K + eps): the product of rows whose RMS norm

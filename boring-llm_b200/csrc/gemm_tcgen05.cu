@@ -172,10 +172,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 uint32_t u[32];
                 tmem_ld32(lane_addr + 64 + c * 32, u);
                 tmem_ld_wait();
-                if (glu.kind == BL_GLU_SILU) {                                  // one branch a chunk, the loops as they were
+                if (glu.kind == BL_GLU_SILU && !glu.bias) {                                  // one branch a chunk, the loops as they were
 #pragma unroll
                     for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(bl_silu_fast(__uint_as_float(r[j])) * __uint_as_float(u[j]));
                 } else {
+                    if (glu.bias) {                                             // (every lane reads the same column's two numbers)
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) {
+                            const int n = min(n0 + c * 32 + j, N - 1);
+                            r[j] = __float_as_uint(__uint_as_float(r[j]) + glu.bias[n]);
+                            u[j] = __float_as_uint(__uint_as_float(u[j]) + glu.bias[N + n]);
+                        }
+                    }
 #pragma unroll
                     for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(bl_glu_fast(glu.kind, __uint_as_float(r[j]), __uint_as_float(u[j]), glu.limit));
                 }
@@ -195,7 +203,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 float4 v = *reinterpret_cast<const float4*>(tile + row * PITCH + c4);
                 TO* dst = out + (size_t)m * N + n;
                 if (vec_ok && n + 3 < N) {
-                    if (EPI == BL_EPI_BIAS) {
+                    if (EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) {
                         v.x += bl_load_any(bias, bias_dtype, n); v.y += bl_load_any(bias, bias_dtype, n + 1);
                         v.z += bl_load_any(bias, bias_dtype, n + 2); v.w += bl_load_any(bias, bias_dtype, n + 3);
                     }
@@ -217,7 +225,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     for (int j = 0; j < 4; ++j) {
                         if (n + j >= N) break;
                         float x1 = e[j];
-                        if (EPI == BL_EPI_BIAS) x1 += bl_load_any(bias, bias_dtype, n + j);
+                        if (EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) x1 += bl_load_any(bias, bias_dtype, n + j);
                         if (EPI == BL_EPI_RESIDUAL) x1 += bl_load(dst + j);
                         bl_store(dst + j, x1);
                     }

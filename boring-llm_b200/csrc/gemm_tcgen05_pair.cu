@@ -380,9 +380,16 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     uint32_t u[32];
                     tmem_ld32(lane_addr + BN / 2 + c * 32, u);
                     tmem_ld_wait();
-                    if (glu.kind == BL_GLU_SILU) {                              // one branch a chunk, the loops as they were
+                    if (glu.kind == BL_GLU_SILU && !glu.bias) {                              // one branch a chunk, the loops as they were
 #pragma unroll
                         for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(bl_silu_fast(__uint_as_float(r[j]) * row_scale) * (__uint_as_float(u[j]) * row_scale));
+                    } else if (glu.bias) {                                      // (every lane reads the same column's two numbers)
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) {
+                            const int n = min(n0 + c * 32 + j, N - 1);
+                            r[j] = __float_as_uint(bl_glu_fast(glu.kind, __uint_as_float(r[j]) * row_scale + glu.bias[n],
+                                                               __uint_as_float(u[j]) * row_scale + glu.bias[N + n], glu.limit));
+                        }
                     } else {
 #pragma unroll
                         for (int j = 0; j < 32; ++j)
@@ -396,7 +403,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     *reinterpret_cast<uint4*>(tile + lane * PITCH + 4 * j) = make_uint4(r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
                 __syncwarp();
                 float4 b4 = make_float4(0.f, 0.f, 0.f, 0.f);              // a lane writes the same four columns in all eight rows
-                if (EPI == BL_EPI_BIAS && vec_ok && n0 + c * 32 + c4 + 3 < N) {
+                if ((EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) && vec_ok && n0 + c * 32 + c4 + 3 < N) {
                     const int n = n0 + c * 32 + c4;
                     b4 = make_float4(bl_load_any(bias, bias_dtype, n), bl_load_any(bias, bias_dtype, n + 1),
                                      bl_load_any(bias, bias_dtype, n + 2), bl_load_any(bias, bias_dtype, n + 3));
@@ -417,7 +424,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     float4 v = *reinterpret_cast<const float4*>(tile + row * PITCH + c4);
                     TO* dst = out + (size_t)m * N + n;
                     if (vec_ok && n + 3 < N) {
-                        if (EPI == BL_EPI_BIAS) { v.x += b4.x; v.y += b4.y; v.z += b4.z; v.w += b4.w; }
+                        if (EPI == BL_EPI_BIAS || EPI == BL_EPI_RESIDUAL) { v.x += b4.x; v.y += b4.y; v.z += b4.z; v.w += b4.w; }
                         if (sizeof(TO) == 4) {
                             if (EPI == BL_EPI_RESIDUAL) { v.x += res[it2].x; v.y += res[it2].y; v.z += res[it2].z; v.w += res[it2].w; }
                             if (link) {
@@ -440,7 +447,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         for (int j = 0; j < 4; ++j) {
                             if (n + j >= N) break;
                             float x1 = e[j];
-                            if (EPI == BL_EPI_BIAS) x1 += bl_load_any(bias, bias_dtype, n + j);
+                            if (EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) x1 += bl_load_any(bias, bias_dtype, n + j);
                             if (EPI == BL_EPI_RESIDUAL) x1 += bl_load(dst + j);
                             bl_store(dst + j, x1);
                         }
@@ -580,7 +587,7 @@ extern "C" int bl_gemm_tc_pair_norm_parts(int M, int N) {
 // bl_gemm_tc_pair_norm_parts(M, N)). A product that takes hw as its x and scales its rows by
 // 1 / sqrt(sum(ss[m, :]) / N + eps) computes what it would from the normed rows. N must be a multiple of 4.
 extern "C" int bl_gemm_tc_pair_residual_norm(const void* x, const void* w, void* out, int M, int N, int K, const void* norm_w,
-                                             int norm_w_dtype, void* hw, float* ss, void* stream) {
+                                             int norm_w_dtype, void* hw, float* ss, const void* bias, int bias_dtype, void* stream) {
     if (M <= 0) return 0;
     if (N <= 0 || K <= 0 || N % 4 != 0) BL_FAIL("bl_gemm_tc_pair_residual_norm: bad sizes N=%d K=%d (N a multiple of 4)", N, K);
     if (K % 8 != 0) BL_FAIL("bl_gemm_tc_pair_residual_norm: K=%d is not a multiple of 8", K);
@@ -589,7 +596,7 @@ extern "C" int bl_gemm_tc_pair_residual_norm(const void* x, const void* w, void*
         BL_FAIL("bl_gemm_tc_pair_residual_norm: needs the norm's weight (float32 or bfloat16), hw and ss");
     NormLink nl = NormLink();
     nl.norm_w = norm_w; nl.norm_w_dtype = norm_w_dtype; nl.hw = (__nv_bfloat16*)hw; nl.ss_out = ss;
-    return launch<BL_EPI_RESIDUAL, float>(x, w, nullptr, 0, out, M, N, K, (cudaStream_t)stream, nl);
+    return launch<BL_EPI_RESIDUAL, float>(x, w, bias, bias_dtype, out, M, N, K, (cudaStream_t)stream, nl);
 }
 
 // out[M, N] (bfloat16) = silu(r g) * (r u) with g, u = hw . Wg^T, hw . Wu^T and r[m] = 1 / sqrt(sum(ss[m, :parts]) * inv_dim + eps):

@@ -213,7 +213,7 @@ gemm_tc_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
             if (n >= N) continue;
             TO* dst = out + (size_t)m * N + n;
             if (vec_ok && n + 3 < N) {
-                if (EPI == BL_EPI_BIAS) {
+                if (EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) {
                     v.x += bl_load_any(bias, bias_dtype, n); v.y += bl_load_any(bias, bias_dtype, n + 1);
                     v.z += bl_load_any(bias, bias_dtype, n + 2); v.w += bl_load_any(bias, bias_dtype, n + 3);
                 }
@@ -235,7 +235,7 @@ gemm_tc_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
                 for (int j = 0; j < 4; ++j) {
                     if (n + j >= N) break;
                     float x1 = e[j];
-                    if (EPI == BL_EPI_BIAS) x1 += bl_load_any(bias, bias_dtype, n + j);
+                    if (EPI == BL_EPI_BIAS || (EPI == BL_EPI_RESIDUAL && bias != nullptr)) x1 += bl_load_any(bias, bias_dtype, n + j);
                     if (EPI == BL_EPI_RESIDUAL) x1 += bl_load(dst + j);
                     bl_store(dst + j, x1);
                 }

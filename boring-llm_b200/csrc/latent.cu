@@ -7,7 +7,7 @@
 //   bl_latent_prep          RMS norms of the query latent and of the key/value latent, rotation of the shared key part,
 //                           the write of [latent | rotated part] into the token's page
 //   bl_head_gemm_plain      a product per head, out[t, h, :] = x[t, h, :] . W_h (strides say how W_h lies), optionally
-//                           times the sigmoid of a gate per output
+//                           times the sigmoid of a gate per output or per head
 //   bl_rope_heads           rotation of a slice of every head of a row (pairs (j, j + half)), cos and sin times a factor
 //   bl_latent_attention_plain   one warp per (token, head) over the cached rows, a window, a sink per head
 // Norm statistics, angles, scores, the softmax and all sums are 32-bit; angle = float(position) * inv_freq[j].
@@ -74,7 +74,7 @@ template <typename TW>
 __global__ void __launch_bounds__(THREADS)
 head_gemm_plain_kernel(const void* x, int x_dtype, size_t ldx, size_t x_head, const TW* __restrict__ w, size_t w_head, size_t w_n,
                        size_t w_k, void* out, int out_dtype, size_t ld_out, size_t out_head, int N, int K, const float* gate,
-                       size_t ld_gate) {
+                       size_t ld_gate, int gate_heads) {
     bl_pdl_trigger();
     bl_pdl_wait();
     extern __shared__ float xs[];
@@ -86,7 +86,7 @@ head_gemm_plain_kernel(const void* x, int x_dtype, size_t ldx, size_t x_head, co
     const TW* wr = w + (size_t)h * w_head + (size_t)n * w_n;
     float acc = 0.f;
     for (int k = 0; k < K; ++k) acc = fmaf(xs[k], bl_load(wr + (size_t)k * w_k), acc);
-    if (gate) acc *= 1.0f / (1.0f + expf(-gate[(size_t)t * ld_gate + (size_t)h * N + n]));
+    if (gate) acc *= 1.0f / (1.0f + expf(-gate[(size_t)t * ld_gate + (gate_heads ? (size_t)h : (size_t)h * N + n)]));
     const size_t o = (size_t)t * ld_out + (size_t)h * out_head + n;
     if (out_dtype == BL_F32) ((float*)out)[o] = acc;
     else ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(acc);
@@ -209,10 +209,11 @@ __global__ void head_tiles_kernel(int* __restrict__ tile, int n, int per) {
     if (i < n) tile[i] = i / per;
 }
 
-// out[t, h * N + n] = hv[h, t, n] * sigmoid(gate[t, h * N + n]): head-major 32-bit sums back to token rows, gated.
+// out[t, h * N + n] = hv[h, t, n] * sigmoid(gate[t, h * N + n]) (gate_heads: gate[t, h]): head-major 32-bit sums back to
+// token rows, gated.
 template <typename TO>
 __global__ void heads_gate_rows_kernel(const float* __restrict__ hv, const float* gate, size_t ld_gate, TO* __restrict__ out, int T, int H,
-                                       int N, size_t Tp) {
+                                       int N, size_t Tp, int gate_heads) {
     bl_pdl_trigger();
     bl_pdl_wait();
     const size_t total = (size_t)T * H * N;
@@ -220,7 +221,7 @@ __global__ void heads_gate_rows_kernel(const float* __restrict__ hv, const float
         const size_t t = e / ((size_t)H * N), c = e % ((size_t)H * N);
         const size_t h = c / N, n = c % N;
         float v = hv[(h * Tp + t) * N + n];
-        if (gate) v *= 1.0f / (1.0f + expf(-gate[t * ld_gate + c]));
+        if (gate) v *= 1.0f / (1.0f + expf(-gate[t * ld_gate + (gate_heads ? h : c)]));
         bl_store(out + e, v);
     }
 }
@@ -236,14 +237,14 @@ extern "C" int bl_head_tiles(int* tile, int n_heads, int per, void* stream) {
 }
 
 extern "C" int bl_heads_gate_rows(const float* hv, const float* gate, long long ld_gate, void* out, int out_dtype, int T, int H, int N,
-                                  int Tp, void* stream) {
+                                  int Tp, int gate_heads, void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || N <= 0 || Tp < T) BL_FAIL("bl_heads_gate_rows: bad sizes T=%d H=%d N=%d Tp=%d", T, H, N, Tp);
     cudaStream_t s = (cudaStream_t)stream;
     const long long total = (long long)T * H * N;
     const int g = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-    if (out_dtype == BL_F32) BL_CUDA(bl_launch_dependent(heads_gate_rows_kernel<float>, dim3(g), dim3(256), 0, s, hv, gate, (size_t)ld_gate, (float*)out, T, H, N, (size_t)Tp));
-    else if (out_dtype == BL_BF16) BL_CUDA(bl_launch_dependent(heads_gate_rows_kernel<__nv_bfloat16>, dim3(g), dim3(256), 0, s, hv, gate, (size_t)ld_gate, (__nv_bfloat16*)out, T, H, N, (size_t)Tp));
+    if (out_dtype == BL_F32) BL_CUDA(bl_launch_dependent(heads_gate_rows_kernel<float>, dim3(g), dim3(256), 0, s, hv, gate, (size_t)ld_gate, (float*)out, T, H, N, (size_t)Tp, gate_heads));
+    else if (out_dtype == BL_BF16) BL_CUDA(bl_launch_dependent(heads_gate_rows_kernel<__nv_bfloat16>, dim3(g), dim3(256), 0, s, hv, gate, (size_t)ld_gate, (__nv_bfloat16*)out, T, H, N, (size_t)Tp, gate_heads));
     else BL_FAIL("bl_heads_gate_rows: unknown dtype %d", out_dtype);
     BL_CHECK_LAUNCH("bl_heads_gate_rows");
     return 0;
@@ -272,7 +273,8 @@ extern "C" int bl_latent_prep(const float* proj, int ld, int off_q, int q_rank, 
 
 extern "C" int bl_head_gemm_plain(const void* x, int x_dtype, long long ldx, long long x_head, const void* w, int w_dtype,
                                   long long w_head, long long w_n, long long w_k, void* out, int out_dtype, long long ld_out,
-                                  long long out_head, int T, int H, int N, int K, const float* gate, long long ld_gate, void* stream) {
+                                  long long out_head, int T, int H, int N, int K, const float* gate, long long ld_gate, int gate_heads,
+                                  void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || N <= 0 || K <= 0 || K > 12000) BL_FAIL("bl_head_gemm_plain: bad sizes H=%d N=%d K=%d", H, N, K);
     if (H > 65535 || T > 65535) BL_FAIL("bl_head_gemm_plain: %d heads and %d rows exceed the grid", H, T);
@@ -282,7 +284,7 @@ extern "C" int bl_head_gemm_plain(const void* x, int x_dtype, long long ldx, lon
     const dim3 grid((N + THREADS - 1) / THREADS, H, T);
     const size_t smem = (size_t)K * sizeof(float);
 #define BL_GO(TW) BL_CUDA(bl_launch_dependent(head_gemm_plain_kernel<TW>, grid, dim3(THREADS), smem, s, x, x_dtype, (size_t)ldx, (size_t)x_head, \
-        (const TW*)w, (size_t)w_head, (size_t)w_n, (size_t)w_k, out, out_dtype, (size_t)ld_out, (size_t)out_head, N, K, gate, (size_t)ld_gate))
+        (const TW*)w, (size_t)w_head, (size_t)w_n, (size_t)w_k, out, out_dtype, (size_t)ld_out, (size_t)out_head, N, K, gate, (size_t)ld_gate, gate_heads))
     if (w_dtype == BL_F32) BL_GO(float);
     else if (w_dtype == BL_BF16) BL_GO(__nv_bfloat16);
     else BL_FAIL("bl_head_gemm_plain: unknown weight dtype %d", w_dtype);

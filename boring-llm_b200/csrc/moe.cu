@@ -1,6 +1,7 @@
 // Routed experts: the choice of experts per token, matrix products whose rows each use the matrix of their own expert, and
 // the weighted sum of a token's expert results.
-//   scores s = sigmoid(z), or softmax(z) over all experts (z: the router's 32-bit logits); choice scores c = s + correction;
+//   scores s = sigmoid(z), or softmax(z) over all experts, or z itself, whose softmax over the CHOSEN experts then gives the
+//   weights (z: the router's 32-bit logits); choice scores c = s + correction;
 //   the experts are n_groups equal runs of neighbours, a group's score is the sum of its two largest choice scores (its only
 //   one where groups hold one expert) or its largest alone, only experts of the `keep` best groups can be chosen; the `top`
 //   largest choice scores among them are chosen (ties: the lower index); the weights are the chosen experts' s, as they are.
@@ -23,7 +24,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
     }
 }
 
-// One warp per token. Shared memory: s [E], c [E], group scores [n_groups], kept flags [n_groups].
+// One warp per token. Shared memory: s [E], c [E], group scores [n_groups], kept flags [n_groups], chosen logits [top].
 __global__ void __launch_bounds__(32)
 moe_route_kernel(const float* __restrict__ z, int ldz, const void* __restrict__ corr, int corr_dtype, int E, int top, int n_groups,
                  int keep, int* __restrict__ ids, float* __restrict__ wts, int score_kind, int group_top) {
@@ -34,6 +35,7 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const void* __restrict__ 
     float* c = sm + E;
     float* gs = sm + 2 * E;
     float* kept = gs + n_groups;
+    float* picked = kept + n_groups;                           // the chosen logits [top] (BL_SCORE_CHOSEN)
     const int t = blockIdx.x, lane = threadIdx.x;
     const int per = E / n_groups;
     float zmax = -INFINITY, zsum = 1.f;
@@ -46,7 +48,7 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const void* __restrict__ 
     }
     for (int e = lane; e < E; e += 32) {
         const float ze = z[(size_t)t * ldz + e];
-        const float v = score_kind == BL_SCORE_SOFTMAX ? expf(ze - zmax) / zsum : 1.0f / (1.0f + expf(-ze));
+        const float v = score_kind == BL_SCORE_CHOSEN ? ze : (score_kind == BL_SCORE_SOFTMAX ? expf(ze - zmax) / zsum : 1.0f / (1.0f + expf(-ze)));
         s[e] = v;
         c[e] = v + (corr ? bl_load_any(corr, corr_dtype, e) : 0.f);
     }
@@ -80,10 +82,17 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const void* __restrict__ 
         if (bi >= E) bi = 0;                                   // fewer open experts than `top` (refused on the host)
         if (lane == 0) {
             ids[(size_t)t * top + n] = bi;
-            wts[(size_t)t * top + n] = s[bi];
+            if (score_kind == BL_SCORE_CHOSEN) picked[n] = s[bi];
+            else wts[(size_t)t * top + n] = s[bi];
             c[bi] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (score_kind == BL_SCORE_CHOSEN) {                       // softmax over the chosen logits, added in the order of the choice
+        float m = -INFINITY, sum = 0.f;
+        for (int n = 0; n < top; ++n) m = fmaxf(m, picked[n]);
+        for (int n = 0; n < top; ++n) sum += expf(picked[n] - m);
+        for (int n = lane; n < top; n += 32) wts[(size_t)t * top + n] = expf(picked[n] - m) / sum;
     }
 }
 
@@ -236,11 +245,11 @@ extern "C" int bl_moe_route(const float* z, int ldz, const void* correction, int
 extern "C" int bl_moe_route_ext(const float* z, int ldz, const void* correction, int corr_dtype, int T, int E, int top, int n_groups,
                                 int keep, int* ids, float* wts, int score_kind, int group_top, void* stream) {
     if (T <= 0) return 0;
-    if ((score_kind != BL_SCORE_SIGMOID && score_kind != BL_SCORE_SOFTMAX) || (group_top != 1 && group_top != 2))
+    if ((score_kind != BL_SCORE_SIGMOID && score_kind != BL_SCORE_SOFTMAX && score_kind != BL_SCORE_CHOSEN) || (group_top != 1 && group_top != 2))
         BL_FAIL("bl_moe_route: scores of kind %d, groups scored by their %d largest", score_kind, group_top);
     if (E <= 0 || top <= 0 || n_groups <= 0 || keep <= 0 || E % n_groups != 0 || keep > n_groups || top > keep * (E / n_groups) || ldz < E)
         BL_FAIL("bl_moe_route: %d experts in %d groups, %d groups kept, %d chosen", E, n_groups, keep, top);
-    const size_t smem = (size_t)(2 * E + 2 * n_groups) * sizeof(float);
+    const size_t smem = (size_t)(2 * E + 2 * n_groups + top) * sizeof(float);
     if (smem > 48 * 1024) BL_FAIL("bl_moe_route: %d experts are too many for shared memory", E);
     BL_CUDA(bl_launch_dependent(moe_route_kernel, dim3(T), dim3(32), smem, (cudaStream_t)stream, z, ldz, correction, corr_dtype, E, top,
                                 n_groups, keep, ids, wts, score_kind, group_top));

@@ -155,20 +155,25 @@ def add_row_vector(x: torch.Tensor, v: torch.Tensor) -> None:
     _call(_lib().bl_add_row_vector, _p(x), _p(v), _dt(v), rows, d, _stream())
 
 
-def glu_args(kind: int, limit: float, device) -> Optional[torch.Tensor]:
+def glu_args(kind: int, limit: float, device, gate_bias: Optional[torch.Tensor] = None,
+             up_bias: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """What a product with the gated epilogue (EPI_SWIGLU) takes in the place of a bias to compute another gated activation
-    than SiLU: the two 32-bit numbers {kind, limit} on the device (GLU_GELU_TANH, GLU_CLAMPED with its limit). None for SiLU."""
+    than SiLU: the two 32-bit numbers {kind, limit} on the device (GLU_GELU_TANH, GLU_CLAMPED with its limit). None for SiLU.
+    `gate_bias` / `up_bias` [N]: biases that the two sums get before the activation; they follow four leading numbers."""
+    if kind not in (GLU_SILU, GLU_GELU_TANH, GLU_CLAMPED):
+        raise KernelError(f"glu_args: unknown gated activation {kind}")
+    if gate_bias is not None or up_bias is not None:
+        head = torch.tensor([float(kind + GLU_BIASED), float(limit), 0.0, 0.0], dtype=torch.float32, device=device)
+        return torch.cat([head, gate_bias.to(head), up_bias.to(head)]).contiguous()
     if kind == GLU_SILU:
         return None
-    if kind not in (GLU_GELU_TANH, GLU_CLAMPED):
-        raise KernelError(f"glu_args: unknown gated activation {kind}")
     return torch.tensor([float(kind), float(limit)], dtype=torch.float32, device=device)
 
 
 def _need_bias(bias: torch.Tensor, N: int, epilogue: int) -> None:
-    """A bias of N values; with the gated epilogue, which adds none, the two numbers of `glu_args`."""
+    """A bias of N values; with the gated epilogue the numbers of `glu_args`."""
     if epilogue == EPI_SWIGLU:
-        _need(bias, "activation", torch.float32, (2,))
+        _need(bias, "activation", torch.float32, (2,) if bias.numel() == 2 else (4 + 2 * N,))
     else:
         _need(bias, "bias", None, (N,))
 
@@ -705,8 +710,9 @@ def gemm_skinny_links_norm(x: torch.Tensor, w: torch.Tensor, N: int, epilogue: i
             and gemm_kernel(x, w, N, None, epilogue, fast) == "skinny")
 
 
-def gemm_skinny_residual_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, norm_w: torch.Tensor):
-    """out += x @ w.T (32-bit residual stream, in place) on the register-streaming kernel, and, for the RMS norm with
+def gemm_skinny_residual_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, norm_w: torch.Tensor,
+                              bias: Optional[torch.Tensor] = None):
+    """out += x @ w.T (+ bias) (32-bit residual stream, in place) on the register-streaming kernel, and, for the RMS norm with
     weight `norm_w` that reads `out` next, (hw, ss): hw = bfloat16(out * norm_w), ss[m, :] = sums of squares of row m
     by block of 16 columns (what `gemm_residual_norm` gives on pairs of SMs, for decode steps)."""
     M, K = x.shape
@@ -716,7 +722,10 @@ def gemm_skinny_residual_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tenso
     parts = int(_lib().bl_gemm_skinny_norm_parts(N))
     hw = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     ss = torch.empty((M, parts), dtype=torch.float32, device=x.device)
-    _call(_lib().bl_gemm_skinny_residual_norm, _p(x), _p(w), _p(out), M, N, K, _p(norm_w), _dt(norm_w), _p(hw), _p(ss), _stream())
+    if bias is not None:
+        _need_bias(bias, N, EPI_RESIDUAL)
+    _call(_lib().bl_gemm_skinny_residual_norm, _p(x), _p(w), _p(out), M, N, K, _p(norm_w), _dt(norm_w), _p(hw), _p(ss), _p(bias),
+          _vec_dt(bias), _stream())
     return hw, ss
 
 
@@ -736,8 +745,8 @@ def gemm_skinny_scaled(hw: torch.Tensor, w: torch.Tensor, out: torch.Tensor, ss:
           M, N, K, epilogue, _p(ss), ss.shape[1], ctypes.c_float(eps), _stream())
 
 
-def gemm_residual_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, norm_w: torch.Tensor):
-    """out += x @ w.T (32-bit residual stream, in place) on pairs of SMs, and, for the RMS norm with weight `norm_w`
+def gemm_residual_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, norm_w: torch.Tensor, bias: Optional[torch.Tensor] = None):
+    """out += x @ w.T (+ bias) (32-bit residual stream, in place) on pairs of SMs, and, for the RMS norm with weight `norm_w`
     that reads `out` next, (hw, ss): hw = bfloat16(out * norm_w) and ss[m, :] = sums of squares of row m's columns by
     tile. A product that takes hw as its x and scales its rows by 1 / sqrt(ss[m].sum() / N + eps) computes what it would
     from the normed rows (`gemm_swiglu_scaled`, `qkv_rope_tc` with `row_sums`)."""
@@ -748,7 +757,10 @@ def gemm_residual_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, norm
     parts = int(_lib().bl_gemm_tc_pair_norm_parts(M, N))
     hw = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     ss = torch.empty((M, parts), dtype=torch.float32, device=x.device)
-    _call(_lib().bl_gemm_tc_pair_residual_norm, _p(x), _p(w), _p(out), M, N, K, _p(norm_w), _dt(norm_w), _p(hw), _p(ss), _stream())
+    if bias is not None:
+        _need_bias(bias, N, EPI_RESIDUAL)
+    _call(_lib().bl_gemm_tc_pair_residual_norm, _p(x), _p(w), _p(out), M, N, K, _p(norm_w), _dt(norm_w), _p(hw), _p(ss), _p(bias),
+          _vec_dt(bias), _stream())
     return hw, ss
 
 
@@ -1284,13 +1296,14 @@ def bonus_dot(q: torch.Tensor, k: torch.Tensor, u: torch.Tensor, out: torch.Tens
     _call(_lib().bl_bonus_dot, _p(q), ldq, _p(k), ldk, _p(u), _dt(u), _p(out), T, H, dk, _stream())
 
 
-SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
+SCORE_SIGMOID, SCORE_SOFTMAX, SCORE_CHOSEN = 0, 1, 2
 
 
 def moe_route(z: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_groups: int, keep: int, ids: torch.Tensor,
               wts: torch.Tensor, score: int = SCORE_SIGMOID, group_top: int = 2) -> None:
     """The experts of each token and their weights from the router's 32-bit logits z [T, E] (see `bl_moe_route`). `score`:
-    sigmoid of each logit, or the softmax over all E; `group_top`: a group's score is the sum of its two largest choice
+    sigmoid of each logit, the softmax over all E, or (SCORE_CHOSEN) the logit itself for the choice and the softmax over the
+    chosen logits alone for the weights; `group_top`: a group's score is the sum of its two largest choice
     scores (2) or its largest (1)."""
     T, E = z.shape
     ld = _rows32(z, "z", T, E)
@@ -1397,6 +1410,7 @@ def moe_combine_rows(y: torch.Tensor, pos: torch.Tensor, wts: torch.Tensor, out:
 
 
 GLU_SILU, GLU_GELU_TANH, GLU_CLAMPED = 0, 1, 2
+GLU_BIASED = 16
 
 
 def glu_act(sums: torch.Tensor, out: torch.Tensor, kind: int, limit: float = 0.0) -> None:
@@ -1452,20 +1466,21 @@ def _head_view(t: torch.Tensor, name: str, T: int, H: int, n: int):
     return t.stride(0), t.stride(1)
 
 
-def head_gemm_plain(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
-    """out[t, h, n] = sum_k x[t, h, k] * w[h, n, k] (times sigmoid(gate[t, h * N + n]) if given): a product per head on
+def head_gemm_plain(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
+                    gate_heads: bool = False) -> None:
+    """out[t, h, n] = sum_k x[t, h, k] * w[h, n, k] (times sigmoid(gate[t, h * N + n]) if given; `gate_heads`: sigmoid(gate[t, h])): a product per head on
     CUDA cores, one FMA chain per output in ascending k. x [T, H, K] and out [T, H, N] are views with a contiguous last
-    dimension (32-bit or bfloat16), w [H, N, K] a view with any strides; gate 32-bit rows [T, >= H * N]."""
+    dimension (32-bit or bfloat16), w [H, N, K] a view with any strides; gate 32-bit rows [T, >= H * N] ([T, >= H])."""
     T, H, K = x.shape
     N = w.shape[1]
     ldx, xh = _head_view(x, "x", T, H, K)
     ldo, oh = _head_view(out, "out", T, H, N)
     if w.dim() != 3 or w.shape[0] != H or w.shape[2] != K or not w.is_cuda:
         raise KernelError(f"head_gemm_plain: w {tuple(w.shape)} does not fit x {tuple(x.shape)}")
-    ld_gate = _rows32(gate, "gate", T, H * N) if gate is not None else 0
+    ld_gate = _rows32(gate, "gate", T, H if gate_heads else H * N) if gate is not None else 0
     _call(_lib().bl_head_gemm_plain, _p(x), _dt(x), ctypes.c_longlong(ldx), ctypes.c_longlong(xh), _p(w), _dt(w),
           ctypes.c_longlong(w.stride(0)), ctypes.c_longlong(w.stride(1)), ctypes.c_longlong(w.stride(2)), _p(out), _dt(out),
-          ctypes.c_longlong(ldo), ctypes.c_longlong(oh), T, H, N, K, _p(gate), ctypes.c_longlong(ld_gate), _stream())
+          ctypes.c_longlong(ldo), ctypes.c_longlong(oh), T, H, N, K, _p(gate), ctypes.c_longlong(ld_gate), 1 if gate_heads else 0, _stream())
 
 
 def rope_heads(q: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, rot_half: int, mscale: float,
@@ -1565,14 +1580,113 @@ def head_tiles(n_heads: int, per: int, device) -> torch.Tensor:
     return tile
 
 
-def heads_gate_rows(hv: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor) -> None:
-    """out[t, h * N + n] = hv[h, t, n] (* sigmoid(gate[t, h * N + n])): head-major 32-bit sums hv [H, Tp, N] back to the
-    step's token rows out [T, H * N]; gate 32-bit rows [T, >= H * N] that may be a column range of a wider matrix."""
+def heads_gate_rows(hv: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, gate_heads: bool = False) -> None:
+    """out[t, h * N + n] = hv[h, t, n] (* sigmoid(gate[t, h * N + n]), or with `gate_heads` sigmoid(gate[t, h])): head-major 32-bit sums hv [H, Tp, N] back to the
+    step's token rows out [T, H * N]; gate 32-bit rows [T, >= H * N] ([T, >= H]) that may be a column range of a wider matrix."""
     H, Tp, N = hv.shape
     T = out.shape[0]
     _need(hv, "hv", torch.float32); _need(out, "out", None, (T, H * N))
-    ld = _rows32(gate, "gate", T, H * N) if gate is not None else 0
-    _call(_lib().bl_heads_gate_rows, _p(hv), _p(gate), ctypes.c_longlong(ld), _p(out), _dt(out), T, H, N, Tp, _stream())
+    ld = _rows32(gate, "gate", T, H if gate_heads else H * N) if gate is not None else 0
+    _call(_lib().bl_heads_gate_rows, _p(hv), _p(gate), ctypes.c_longlong(ld), _p(out), _dt(out), T, H, N, Tp, 1 if gate_heads else 0,
+          _stream())
+
+
+def concat_rows(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t] = [a[t] | b[t]] in out's dtype: 32-bit rows [T, m] and [T, n] side by side."""
+    T, m = a.shape
+    n = b.shape[1]
+    _need(a, "a", torch.float32); _need(b, "b", torch.float32, (T, n)); _need(out, "out", None, (T, m + n))
+    _call(_lib().bl_concat_rows, _p(a), m, _p(b), n, _p(out), _dt(out), T, _stream())
+
+
+# ---- attention whose heads' scores are mixed before the softmax --------------------------------------------------------------
+MIXED_MAX_SPLITS = 16          # slices of a single token's keys: the blocks of one cluster
+_mixed_resident = {}
+
+
+def _rms_cache(k_rms: torch.Tensor, k_cache: torch.Tensor):
+    """(pointer, floats between entries) of the keys' root mean squares: pages [pages, KV, page, 2] of the cache's dtype whose
+    entries hold one 32-bit number (two bfloat16 places, or the first of two 32-bit ones)."""
+    if tuple(k_rms.shape) != tuple(k_cache.shape[:3]) + (2,) or k_rms.dtype != k_cache.dtype or not k_rms.is_contiguous():
+        raise KernelError(f"k_rms: must be contiguous {tuple(k_cache.shape[:3]) + (2,)} {k_cache.dtype}, got {tuple(k_rms.shape)} {k_rms.dtype}")
+    return _p(k_rms), 1 if k_rms.dtype == torch.bfloat16 else 2
+
+
+def mixed_prep(proj: torch.Tensor, off_k: int, talk: torch.Tensor, eps: float, positions: torch.Tensor, tok_req: torch.Tensor,
+               block_table: torch.Tensor, q_out: torch.Tensor, k_cache: Optional[torch.Tensor], k_rms: Optional[torch.Tensor]) -> None:
+    """From the 32-bit rows proj (q from column 0, k from off_k): q_out[t, h, c] = sum_{g of key/value head c} talk[h, g] *
+    (q_g / rms(q_g)), keys / rms into the pages, their rms beside them (None, None: the cache is not written)."""
+    T, H, KV, dh = q_out.shape
+    ld = _rows32(proj, "proj", T, off_k + KV * dh)
+    _need(talk, "talk", torch.float32, (H, H)); _need(q_out, "q_out"); _need(positions, "positions", torch.int32, (T,))
+    _need(tok_req, "tok_req", torch.int32, (T,)); _need(block_table, "block_table", torch.int32)
+    page, rms, stride = 16, None, 1
+    if k_cache is not None:
+        _need(k_cache, "k_cache", q_out.dtype)
+        if k_cache.dim() != 4 or k_cache.shape[1] != KV or k_cache.shape[3] != dh:
+            raise KernelError(f"mixed_prep: cache {tuple(k_cache.shape)} does not hold {KV} key heads of {dh}")
+        page = k_cache.shape[2]
+        rms, stride = _rms_cache(k_rms, k_cache)
+    _call(_lib().bl_mixed_prep, _p(proj), ld, off_k, _p(talk), ctypes.c_float(eps), _p(positions), _p(tok_req), _p(block_table),
+          block_table.shape[1], _p(q_out), _p(k_cache), rms, stride, _dt(q_out), T, H, KV, dh, page, _stream())
+
+
+def attention_mixed_supported(dtype: torch.dtype, KV: int, dh: int, page_size: int) -> bool:
+    """Whether the tensor-core kernels take these sizes: bfloat16, pages of 16, head sizes that are multiples of 8 up to 128,
+    queries over all key/value heads that fit shared memory."""
+    return dtype == torch.bfloat16 and bool(_lib().bl_attention_mixed_supported(KV, dh, page_size))
+
+
+def _mixed_args(q, k_cache, cu_q, ctx_len, block_table, out, slopes, gate):
+    T, H, KV, dh = q.shape
+    _need(q, "q", k_cache.dtype); _need(k_cache, "k_cache"); _need(out, "out", q.dtype, (T, H * dh))
+    if k_cache.dim() != 4 or k_cache.shape[1] != KV or k_cache.shape[3] != dh:
+        raise KernelError(f"attention_mixed: cache {tuple(k_cache.shape)} does not hold {KV} key heads of {dh}")
+    _need(cu_q, "cu_q", torch.int32); _need(ctx_len, "ctx_len", torch.int32); _need(block_table, "block_table", torch.int32)
+    if slopes is not None:
+        _need(slopes, "slopes", torch.float32, (H,))
+    return T, H, KV, dh, _rows32(gate, "gate", T, H * dh) if gate is not None else 0
+
+
+def attention_mixed_plain(q, k_cache, k_rms, tok_req, cu_q, ctx_len, block_table, out, scale: float,
+                          slopes: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """Causal attention with the mixed queries q [T, H, KV, dh] (`mixed_prep`): score = q . (the keys of all key/value heads) *
+    scale - slopes[h] * (i - j), softmax, values = the head's own keys times their root mean squares; out [T, H * dh], times
+    sigmoid(gate[t, h * dh + d]) if given (32-bit rows). Plain kernel, any dtype."""
+    T, H, KV, dh, ldg = _mixed_args(q, k_cache, cu_q, ctx_len, block_table, out, slopes, gate)
+    _need(tok_req, "tok_req", torch.int32, (T,))
+    rms, stride = _rms_cache(k_rms, k_cache)
+    _call(_lib().bl_attention_mixed_plain, _p(q), _p(k_cache), rms, stride, _dt(q), _p(tok_req), _p(cu_q), _p(ctx_len), _p(block_table),
+          block_table.shape[1], _p(slopes), _p(gate), ldg, _p(out), T, H, KV, dh, k_cache.shape[2], ctypes.c_float(scale), _stream())
+
+
+def attention_mixed_prefill(q, k_cache, k_rms, cu_q, ctx_len, block_table, tiles, out, scale: float,
+                            slopes: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """The same on tensor cores for the requests with several new tokens (tiles [n, 2]: request, first token of 64)."""
+    T, H, KV, dh, ldg = _mixed_args(q, k_cache, cu_q, ctx_len, block_table, out, slopes, gate)
+    _need(tiles, "tiles", torch.int32); _need(k_cache, "k_cache", torch.bfloat16)
+    _call(_lib().bl_attention_mixed_prefill, _p(q), _p(k_cache), _rms_cache(k_rms, k_cache)[0], _p(cu_q), _p(ctx_len), _p(block_table),
+          block_table.shape[1], _p(tiles), tiles.shape[0], _p(out), H, KV, dh, k_cache.shape[2], ctypes.c_float(scale), _p(slopes),
+          _p(gate), ldg, _stream())
+
+
+def attention_mixed_decode(q, k_cache, k_rms, cu_q, ctx_len, block_table, reqs, n_splits: int, out, scale: float,
+                           slopes: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """The same for the requests with a single new token (reqs [n]), whose keys n_splits blocks share."""
+    T, H, KV, dh, ldg = _mixed_args(q, k_cache, cu_q, ctx_len, block_table, out, slopes, gate)
+    _need(reqs, "reqs", torch.int32); _need(k_cache, "k_cache", torch.bfloat16)
+    _call(_lib().bl_attention_mixed_decode, _p(q), _p(k_cache), _rms_cache(k_rms, k_cache)[0], _p(cu_q), _p(ctx_len), _p(block_table),
+          block_table.shape[1], _p(reqs), reqs.shape[0], n_splits, _p(out), H, KV, dh, k_cache.shape[2], ctypes.c_float(scale), _p(slopes),
+          _p(gate), ldg, _stream())
+
+
+def attention_mixed_splits(n: int, H: int, KV: int, dh: int, longest: int) -> int:
+    """Into how many slices the keys of n single-token requests are cut: as many as fill the device once, 64 keys each at
+    least, at most a cluster of blocks."""
+    key = (torch.cuda.current_device(), KV, dh)
+    if key not in _mixed_resident:
+        _mixed_resident[key] = max(1, int(_lib().bl_attention_mixed_decode_resident_blocks(KV, dh)))
+    return max(1, min(-(-longest // 64), _mixed_resident[key] // max(1, n * (-(-H // 16))), MIXED_MAX_SPLITS))
 
 
 def rope_decay_prep(proj: torch.Tensor, off_k: int, positions: torch.Tensor, inv_freq: torch.Tensor, rot_half: int,

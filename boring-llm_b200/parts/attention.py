@@ -511,6 +511,117 @@ class ChunkedTalkingAttention(Mixer):
         self._run(ctx, h, out, cache_layer, write_cache, EPI_NONE)
 
 
+def distance_slopes(n_heads: int):
+    """2^(-8 (h + 1) / n_heads) for head h: slopes of a score's loss per position of distance."""
+    return [2.0 ** (-8.0 * (h + 1) / n_heads) for h in range(n_heads)]
+
+
+class MixedScoreAttention(Mixer):
+    """Causal grouped-query attention whose heads' SCORES are mixed before the softmax, without a value projection:
+
+    * q and k are divided by their root mean square per head (`qk_norm_eps`, no weights); there is no rotation;
+    * the values are the keys as projected, before that norm (there is no Wv);
+    * score_h = q_h . k_kv(h) * scale - slopes[h] * (i - j) (`slopes`: one number per head, None for no distance bias); then
+      score'_h = sum_g talk[h, g] score_g (`talk` [H, H]), and head h's softmax over j <= i applies to the values of its own
+      key/value head;
+    * `out_gate=True`: the concatenated heads are multiplied by sigmoid(h Wg^T), one number per channel.
+
+    The mix is linear in the query and in the slope, so both are mixed instead of the scores (`ops.mixed_prep`): per head one
+    query over the keys of ALL key/value heads side by side, and one slope. The cache keeps the normed keys and, per
+    (token, key/value head), the root mean square they were divided by: a value is their product, so nothing else is stored
+    (`PagedKVSpec` with values of two places, which hold one 32-bit number). q, k and the gate's logits are ONE joined
+    product with 32-bit sums; norms, mix and cache write are one kernel; the gate is applied where the attention's result is
+    written. Norms, scores, bias, softmax and the root mean squares are 32-bit."""
+    graph_safe = True
+
+    def __init__(self, dim: int, n_heads: int, n_kv_heads: int, head_dim: int, names: Dict[str, str], scale: Optional[float] = None,
+                 qk_norm_eps: float = 1e-6, slopes=None, out_gate: bool = False):
+        super().__init__(names)
+        if n_heads % n_kv_heads != 0:
+            raise ValueError(f"{n_heads} query heads cannot share {n_kv_heads} key/value heads")
+        self.dim, self.H, self.KV, self.dh = dim, n_heads, n_kv_heads, head_dim
+        self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
+        self.qk_norm_eps, self.out_gate = float(qk_norm_eps), bool(out_gate)
+        if slopes is not None and len(slopes) != n_heads:
+            raise ValueError(f"{len(slopes)} slopes for {n_heads} heads")
+        self.slopes_host = [float(s) for s in slopes] if slopes is not None else None
+        pad = lambda n: -(-n // 8) * 8              # every part of the joined product starts on a 32-byte boundary of the sums
+        self.off_k = pad(n_heads * head_dim)
+        self.off_g = self.off_k + pad(n_kv_heads * head_dim)
+        self.n_in = self.off_g + (pad(n_heads * head_dim) if self.out_gate else 0)
+        self.w_in = self.wo = self.talk = self.slopes = None
+
+    def local_specs(self):
+        s = {"wq": TensorSpec((self.H * self.dh, self.dim), MATRIX), "wk": TensorSpec((self.KV * self.dh, self.dim), MATRIX),
+             "wo": TensorSpec((self.dim, self.H * self.dh), MATRIX), "talk": TensorSpec((self.H, self.H), MATRIX)}
+        if self.out_gate:
+            s["wg"] = TensorSpec((self.H * self.dh, self.dim), MATRIX)
+        return s
+
+    def place(self, local, dtype, device):
+        w_in = torch.zeros((self.n_in, self.dim), dtype=local["wq"].dtype, device=local["wq"].device)
+        w_in[:self.H * self.dh] = local["wq"]
+        w_in[self.off_k:self.off_k + self.KV * self.dh] = local["wk"]
+        if self.out_gate:
+            w_in[self.off_g:self.off_g + self.H * self.dh] = local["wg"]
+        self.w_in = to_device_matrix(w_in, dtype, device)
+        self.wo = to_device_matrix(local["wo"], dtype, device)
+        talk = local["talk"].to(torch.float32)
+        self.talk = talk.to(device=device).contiguous()
+        if self.slopes_host is not None:
+            mixed = talk.cpu().to(torch.float64) @ torch.tensor(self.slopes_host, dtype=torch.float64)
+            self.slopes = mixed.to(torch.float32).to(device).contiguous()
+
+    def cache_spec(self):
+        return PagedKVSpec(self.KV, self.dh, 0, 2)
+
+    def takes_pending_norm_at(self, rows: int) -> bool:
+        """As for `LatentAttention`: the joined first product finishes a norm where it runs on the register-streaming kernel."""
+        return (ops.SKINNY_LINK_MIN_ROWS <= rows <= ops.SKINNY_LINK_MAX_ROWS and self.w_in is not None
+                and self.w_in.dtype == torch.bfloat16 and -(-self.n_in // 16) <= ops.SKINNY_LINK_MAX_BLOCKS
+                and not ops.gemm_streams_better(self.w_in))
+
+    def plan_step(self, q_lens, ctx_lens, filler=None):
+        return PLAN_KEY, attention_plan(q_lens, ctx_lens, filler)
+
+    def attend(self, ctx, q, k_cache, k_rms, table, gate, out):
+        """q [T, H, KV, dh] mixed queries; out [T, H * dh]."""
+        if not (ctx.fast and ops.attention_mixed_supported(q.dtype, self.KV, self.dh, k_cache.shape[2])):
+            ops.attention_mixed_plain(q, k_cache, k_rms, ctx.tok_req, ctx.cu_q, ctx.ctx_len, table, out, self.scale, self.slopes, gate)
+            return
+        plan = ctx.plans.get(PLAN_KEY)
+        if plan is None:                                 # a step put together without asking the parts: plan it now
+            plan = attention_plan(ctx.q_lens, ctx.ctx_lens)
+            plan.arrays = {k: torch.from_numpy(v).to(ctx.device) for k, v in plan.arrays.items()}
+            ctx.plans[PLAN_KEY] = plan
+        tiles64, singles = plan.arrays["tiles64"], plan.arrays["singles"]
+        if tiles64.shape[0]:
+            ops.attention_mixed_prefill(q, k_cache, k_rms, ctx.cu_q, ctx.ctx_len, table, tiles64, out, self.scale, self.slopes, gate)
+        n = singles.shape[0]
+        if n:
+            splits = ops.attention_mixed_splits(n, self.H, self.KV, self.dh, plan.host["longest_single"])
+            ops.attention_mixed_decode(q, k_cache, k_rms, ctx.cu_q, ctx.ctx_len, table, singles, splits, out, self.scale, self.slopes, gate)
+
+    def _run(self, ctx, h, out, cache_layer, write_cache, epilogue):
+        T = h.shape[0]
+        k_cache, k_rms, table = ctx.kv(cache_layer)
+        proj = ctx.empty((T, self.w_in.shape[0]), torch.float32)
+        linear(ctx, h, self.w_in, proj, None, EPI_NONE)
+        self._joined(proj)
+        q = ctx.empty((T, self.H, self.KV, self.dh))
+        ops.mixed_prep(proj, self.off_k, self.talk, self.qk_norm_eps, ctx.positions, ctx.tok_req, table, q,
+                       k_cache if write_cache else None, k_rms if write_cache else None)
+        attn = ctx.empty((T, self.H * self.dh))
+        self.attend(ctx, q, k_cache, k_rms, table, proj[:, self.off_g:self.off_g + self.H * self.dh] if self.out_gate else None, attn)
+        linear(ctx, attn, self.wo, out, None, epilogue)
+
+    def forward(self, ctx, h, residual, cache_layer, write_cache=True):
+        self._run(ctx, h, residual, cache_layer, write_cache, EPI_RESIDUAL)
+
+    def mix(self, ctx, h, out, cache_layer, write_cache=True):
+        self._run(ctx, h, out, cache_layer, write_cache, EPI_NONE)
+
+
 class ParallelMixers(Mixer):
     """Two mixers side by side that read the same rows. Each mixer keeps its own cache, so this part's `cache_spec()` is the
     pair of theirs and it is handed a pair of cache layers. How the two results join is `combine`:

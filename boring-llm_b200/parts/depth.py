@@ -6,8 +6,9 @@ from typing import Dict
 import torch
 
 from ..kernels import ops
-from ..weights import TensorSpec, NORM
+from ..weights import TensorSpec, MATRIX, NORM
 from .base import Part
+from .linear import linear, EPI_NONE
 
 
 class DepthWeightedAverage(Part):
@@ -24,6 +25,29 @@ class DepthWeightedAverage(Part):
 
     def forward(self, ctx, streams: torch.Tensor, out: torch.Tensor) -> None:
         ops.depth_mix(streams, self.weight, self.n, out)
+
+
+class StreamReentry(Part):
+    """x <- W [x | x0]: what the first layer of each pass of a loop reads, from the stream x and the embedding rows x0
+    (`weight` [dim, 2 dim], x first). The result is a new 32-bit stream; x0 stays as it is."""
+
+    def __init__(self, dim: int, names: Dict[str, str]):
+        super().__init__(names)
+        self.dim = dim
+        self.weight = None
+
+    def local_specs(self):
+        return {"weight": TensorSpec((self.dim, 2 * self.dim), MATRIX)}
+
+    def forward(self, ctx, x: torch.Tensor, x0: torch.Tensor) -> torch.Tensor:
+        both = ctx.empty((x.shape[0], 2 * self.dim))
+        ops.concat_rows(x, x0, both)
+        out = ctx.empty(tuple(x.shape), torch.float32)
+        after, ctx.next_norm = ctx.next_norm, None       # a fresh stream: no product before it has begun a norm of it
+        ctx.memo.pop(("pending norm", id(out)), None)
+        linear(ctx, both, self.weight, out, None, EPI_NONE)
+        ctx.next_norm = after
+        return out
 
 
 class AfterBlock:

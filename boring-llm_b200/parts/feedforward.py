@@ -7,8 +7,8 @@ import torch
 
 from ..kernels import ops
 from ..weights import TensorSpec, MATRIX, BIAS, INT_TABLE
-from .base import Part, to_device_matrix
-from .linear import linear, EPI_NONE, EPI_RESIDUAL, EPI_SWIGLU
+from .base import Part, to_device_matrix, to_device_vector
+from .linear import linear, EPI_BIAS, EPI_NONE, EPI_RESIDUAL, EPI_SWIGLU
 
 
 FF_FUSED_MAX_ROWS = 16    # more rows: a separate norm and the tcgen05 product are faster (measured: 6% of a step at 24 and 32 rows)
@@ -138,20 +138,22 @@ class SwiGLU(FeedForward):
 
 
 class GluMLP(FeedForward):
-    """down(glu(gate(h), up(h))), no biases, with the gated activation as an argument:
+    """down(glu(gate(h), up(h))) with the gated activation as an argument, and biases on all three products with `bias=True`:
 
     * "silu":       silu(g) * u (what `SwiGLU` computes with fused epilogues);
     * "gelu_tanh":  0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u;
     * "clamped":    g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(1.702 g') (u' + 1).
 
     Gate and up are one joined product over [Wg; Wu] whose epilogue evaluates the activation on the 32-bit sums (the
-    epilogue of `SwiGLU`, told which activation by two numbers on the device); the down product adds into the residual
-    stream."""
+    epilogue of `SwiGLU`, told which activation, and its biases, by numbers on the device); the down product adds into the
+    residual stream, its bias with it."""
     graph_safe = True
     KINDS = {"silu": ops.GLU_SILU, "gelu_tanh": ops.GLU_GELU_TANH, "clamped": ops.GLU_CLAMPED}
 
-    def __init__(self, dim: int, hidden: int, names: Dict[str, str], activation: str = "silu", limit: float = 0.0):
+    def __init__(self, dim: int, hidden: int, names: Dict[str, str], activation: str = "silu", limit: float = 0.0,
+                 bias: bool = False):
         super().__init__(names)
+        self.bias, self.b_down = bool(bias), None
         if activation not in self.KINDS:
             raise ValueError(f"GluMLP: activation must be one of {sorted(self.KINDS)}, got {activation!r}")
         if activation == "clamped" and not limit > 0:
@@ -160,14 +162,20 @@ class GluMLP(FeedForward):
         self.w_gate_up = self.w_down = self.act_args = None
 
     def local_specs(self):
-        return {"w_gate": TensorSpec((self.hidden, self.dim), MATRIX),
-                "w_up": TensorSpec((self.hidden, self.dim), MATRIX),
-                "w_down": TensorSpec((self.dim, self.hidden), MATRIX)}
+        s = {"w_gate": TensorSpec((self.hidden, self.dim), MATRIX),
+             "w_up": TensorSpec((self.hidden, self.dim), MATRIX),
+             "w_down": TensorSpec((self.dim, self.hidden), MATRIX)}
+        if self.bias:
+            s.update({"b_gate": TensorSpec((self.hidden,), BIAS), "b_up": TensorSpec((self.hidden,), BIAS),
+                      "b_down": TensorSpec((self.dim,), BIAS)})
+        return s
 
     def place(self, local, dtype, device):
         self.w_gate_up = to_device_matrix(torch.cat([local["w_gate"], local["w_up"]], dim=0), dtype, device)
         self.w_down = to_device_matrix(local["w_down"], dtype, device)
-        self.act_args = ops.glu_args(self.KINDS[self.activation], self.limit, device)
+        self.act_args = ops.glu_args(self.KINDS[self.activation], self.limit, device, local.get("b_gate"), local.get("b_up"))
+        if self.bias:
+            self.b_down = to_device_vector(local["b_down"], dtype, device)
 
     def takes_pending_norm_at(self, rows: int) -> bool:
         """gate/up finishes a norm that the product before has begun on the register-streaming kernel (a decode step's 2
@@ -181,7 +189,7 @@ class GluMLP(FeedForward):
     def _run(self, ctx, h, out, epilogue):
         act = ctx.empty((h.shape[0], self.hidden))
         linear(ctx, h, self.w_gate_up, act, self.act_args, EPI_SWIGLU)
-        linear(ctx, act, self.w_down, out, None, epilogue)
+        linear(ctx, act, self.w_down, out, self.b_down, EPI_BIAS if self.bias and epilogue == EPI_NONE else epilogue)
 
     def forward(self, ctx, h, residual):
         self._run(ctx, h, residual, EPI_RESIDUAL)
@@ -271,17 +279,19 @@ class RoutedExperts(FeedForward):
     chosen expert) pair is a row of two products whose rows each use the matrix of their own expert. `activation` /
     `limit`: the experts' gated activation, as in `GluMLP`, evaluated in the first product's epilogue.
 
-    Further choices: `score` "sigmoid" or "softmax" (the softmax of z over ALL router outputs); `group_score` "top2" (the sum
+    Further choices: `score` "sigmoid", "softmax" (the softmax of z over ALL router outputs) or "chosen" (the choice runs on z
+    itself, the weights are the softmax over the chosen logits alone); `router_bias`: z = h Wr^T + b; `group_score` "top2" (the sum
     of a group's two largest choice scores) or "max" (its largest); `n_identity`: the router has `n_experts + n_identity`
     outputs, and the last `n_identity` are identity experts without tensors whose output is the input row h itself (times
     the weight); groups are formed over experts and identity experts together."""
     graph_safe = True
-    SCORES = {"sigmoid": ops.SCORE_SIGMOID, "softmax": ops.SCORE_SOFTMAX}
+    SCORES = {"sigmoid": ops.SCORE_SIGMOID, "softmax": ops.SCORE_SOFTMAX, "chosen": ops.SCORE_CHOSEN}
 
     def __init__(self, dim: int, hidden: int, n_experts: int, top: int, names: Dict[str, str], n_groups: int = 1,
                  keep_groups: int = 1, correction: bool = True, activation: str = "silu", limit: float = 0.0,
-                 score: str = "sigmoid", group_score: str = "top2", n_identity: int = 0):
+                 score: str = "sigmoid", group_score: str = "top2", n_identity: int = 0, router_bias: bool = False):
         super().__init__(names)
+        self.has_router_bias, self.b_router = bool(router_bias), None
         if score not in self.SCORES or group_score not in ("top2", "max") or n_identity < 0:
             raise ValueError(f"RoutedExperts: score {score!r}, group_score {group_score!r}, {n_identity} identity experts")
         self.score, self.group_top, self.n_identity = self.SCORES[score], 2 if group_score == "top2" else 1, int(n_identity)
@@ -305,6 +315,8 @@ class RoutedExperts(FeedForward):
         s = {"router": TensorSpec((self.n_out, self.dim), MATRIX)}
         if self.has_correction:
             s["correction"] = TensorSpec((self.n_out,), BIAS)
+        if self.has_router_bias:
+            s["router_bias"] = TensorSpec((self.n_out,), BIAS)
         return s
 
     def local_specs(self):
@@ -319,6 +331,8 @@ class RoutedExperts(FeedForward):
         self.router = to_device_matrix(local["router"], dtype, device)
         if self.has_correction:
             self.correction = local["correction"].to(device=device, dtype=torch.float32).contiguous()
+        if self.has_router_bias:
+            self.b_router = local["router_bias"].to(device=device, dtype=torch.float32).contiguous()
 
     def place(self, local, dtype, device):
         self.place_choice(local, dtype, device)
@@ -334,12 +348,14 @@ class RoutedExperts(FeedForward):
         self.n_own = self.router.shape[0] + pad
         self.router = torch.cat([self.router, self.router.new_zeros((pad, self.router.shape[1])),
                                  weight.to(device=self.router.device, dtype=self.router.dtype)], dim=0).contiguous()
+        if self.b_router is not None:            # (the further rows have no bias)
+            self.b_router = torch.cat([self.b_router, self.b_router.new_zeros(self.router.shape[0] - self.b_router.shape[0])]).contiguous()
 
     def route(self, ctx, h):
         """(experts [T, top] int32, weights [T, top] 32-bit) of the rows h."""
         T = h.shape[0]
         z = ctx.empty((T, self.router.shape[0]), torch.float32)
-        linear(ctx, h, self.router, z, None, EPI_NONE)            # 32-bit sums of exact products (the rows may be bfloat16 roundings)
+        linear(ctx, h, self.router, z, self.b_router, EPI_BIAS if self.has_router_bias else EPI_NONE)     # 32-bit sums of exact products (the rows may be bfloat16 roundings)
         n_own = getattr(self, "n_own", None)
         self.joined_out = z[:, n_own:] if n_own is not None else None
         if n_own is not None:

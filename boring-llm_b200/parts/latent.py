@@ -24,7 +24,10 @@ class LatentAttention(Mixer):
       Uv_h c (`wuk` [H * nope_dim, kv_rank], `wuv` [H * v_dim, kv_rank], head by head);
     * score = (q_nope . k_nope + q_rot . k_rot) * scale; `window` n > 0: position i sees j with 0 <= i - j < n;
       `sink=True`: exp(sink_h) joins head h's softmax denominator once, unscaled, with no value;
-    * `out_gate=True`: the concatenated heads are multiplied by sigmoid(h Wg^T), one number per channel;
+    * `out_gate`: "channel" (or True): the concatenated heads are multiplied by sigmoid(h Wg^T), one number per channel;
+      "head": by one number per head (`wg` [H, dim]);
+    * `rotary`: any `RotaryTable`; interleaved pairs are turned into halves when the weights are placed (the rows that make
+      the rotated parts of q and of the shared key are reordered in the same way, which no score notices);
     * `own_kv=False`: the mixer has no Wdkv and reads the latent and rotated part that another layer cached (its run-order
       entry names that cache layer with `write_cache=False`); `cache_window` is then what the owner and all its readers
       agree the cache keeps (the widest of their windows, 0 if any sees everything).
@@ -45,24 +48,28 @@ class LatentAttention(Mixer):
 
     def __init__(self, dim: int, n_heads: int, nope_dim: int, rot_dim: int, v_dim: int, q_rank: int, kv_rank: int,
                  rotary: Optional[RotaryTable], names: Dict[str, str], window: int = 0, scale: Optional[float] = None,
-                 norm_eps: float = 1e-6, sink: bool = False, out_gate: bool = False, own_kv: bool = True,
+                 norm_eps: float = 1e-6, sink: bool = False, out_gate=False, own_kv: bool = True,
                  cache_window: Optional[int] = None):
         super().__init__(names)
         self.dim, self.H, self.dn, self.dr, self.dv = dim, n_heads, nope_dim, rot_dim, v_dim
         self.q_rank, self.rank = q_rank, kv_rank
         self.rotary = rotary if rotary is not None else RotaryTable(max(rot_dim, 2), 10000.0, n_rot=0)
-        if self.rotary.pairs != "halves" or 2 * self.rotary.rot_half > rot_dim:
+        if 2 * self.rotary.rot_half > rot_dim:
             raise ValueError(f"LatentAttention: the rotation ({self.rotary.n_rot} values in {self.rotary.pairs}) does not fit a rotated part of {rot_dim}")
         self.window = int(window)
         self.cache_window = self.window if cache_window is None else int(cache_window)
         if self.cache_window != 0 and (self.window == 0 or self.window > self.cache_window):
             raise ValueError(f"LatentAttention: a window of {self.window} over a cache that keeps {self.cache_window}")
         self.scale = float(scale) if scale is not None else float(nope_dim + rot_dim) ** -0.5
+        if out_gate not in (False, None, True, "channel", "head"):
+            raise ValueError(f"LatentAttention: out_gate must be 'channel' or 'head', got {out_gate!r}")
+        self.gate_heads = out_gate == "head"
         self.eps, self.has_sink, self.out_gate, self.own_kv = float(norm_eps), bool(sink), bool(out_gate), bool(own_kv)
         pad = lambda n: -(-n // 8) * 8              # every part of the joined product starts on a 32-byte boundary of the sums
         self.off_kv = pad(q_rank)
         self.off_g = self.off_kv + (pad(kv_rank + rot_dim) if self.own_kv else 0)
-        self.n_in = self.off_g + (n_heads * v_dim if self.out_gate else 0)
+        self.n_gate = (n_heads if self.gate_heads else n_heads * v_dim) if self.out_gate else 0
+        self.n_in = self.off_g + (pad(self.n_gate) if self.gate_heads else self.n_gate)
         self.w_in = self.wuq = self.wuk = self.wuv = self.wo = self.dq_norm = self.dkv_norm = self.sinks = None
 
     def local_specs(self):
@@ -76,20 +83,30 @@ class LatentAttention(Mixer):
         if self.has_sink:
             s["sink"] = TensorSpec((self.H,), BIAS)
         if self.out_gate:
-            s["wg"] = TensorSpec((self.H * self.dv, self.dim), MATRIX)
+            s["wg"] = TensorSpec((self.n_gate, self.dim), MATRIX)
         return s
 
+    def _halves(self, w, lead: int):
+        """Rows lead .. of w (the rotated part) with interleaved pairs (2i, 2i + 1) moved to (i, i + half)."""
+        if self.rotary.pair_layout == 0 or not self.rotary.rot_half:
+            return w
+        n = 2 * self.rotary.rot_half
+        order = list(range(lead)) + [lead + i for i in range(0, n, 2)] + [lead + i for i in range(1, n, 2)]
+        return w[order + list(range(lead + n, w.shape[0]))]
+
     def place(self, local, dtype, device):
-        w_in = torch.zeros((self.n_in, self.dim), dtype=local["wdq"].dtype)
+        w_in = torch.zeros((self.n_in, self.dim), dtype=local["wdq"].dtype, device=local["wdq"].device)
         w_in[:self.q_rank] = local["wdq"]
         if self.own_kv:
-            w_in[self.off_kv:self.off_kv + self.rank + self.dr] = local["wdkv"]
+            w_in[self.off_kv:self.off_kv + self.rank + self.dr] = self._halves(local["wdkv"], self.rank)
             self.dkv_norm = to_device_vector(local["dkv_norm"], dtype, device)
         if self.out_gate:
-            w_in[self.off_g:] = local["wg"]
+            w_in[self.off_g:self.off_g + self.n_gate] = local["wg"]
         self.w_in = to_device_matrix(w_in, dtype, device)
         self.dq_norm = to_device_vector(local["dq_norm"], dtype, device)
-        self.wuq = to_device_matrix(local["wuq"], dtype, device)
+        per = self.dn + self.dr
+        wuq = torch.cat([self._halves(local["wuq"][h * per:(h + 1) * per], self.dn) for h in range(self.H)])
+        self.wuq = to_device_matrix(wuq, dtype, device)
         self.wuk = to_device_matrix(local["wuk"], dtype, device)              # [H * nope_dim, kv_rank] as stored
         # Uk_h^T stacked [H, kv_rank, nope_dim]: the matrices of the grouped product that moves the queries into the latent's space
         self.wuk_t = to_device_matrix(local["wuk"].view(self.H, self.dn, self.rank).transpose(1, 2).contiguous(), dtype, device)
@@ -170,7 +187,11 @@ class LatentAttention(Mixer):
                                          self.sinks, splits)
         hv = ctx.empty((H, Tp, self.dv), torch.float32)
         ops.gemm_grouped(lat.view(H * Tp, self.rank), self.wuv.view(H, self.dv, self.rank), tile_head, hv.view(H * Tp, self.dv), EPI_NONE)
-        ops.heads_gate_rows(hv, gate, heads)
+        ops.heads_gate_rows(hv, gate, heads, gate_heads=self.gate_heads)
+
+    def _gate(self, proj):
+        """The gate's logits among the joined product's sums."""
+        return proj[:, self.off_g:self.off_g + self.n_gate] if self.out_gate else None
 
     def _run(self, ctx, h, out, cache_layer, write_cache, epilogue):
         T = h.shape[0]
@@ -185,7 +206,7 @@ class LatentAttention(Mixer):
                         cache if write_cache else None)
         if self.head_major(ctx, cache):
             heads = ctx.empty((T, self.H * self.dv))
-            self._attend_head_major(ctx, cq, cache, table, proj[:, self.off_g:] if self.out_gate else None, heads)
+            self._attend_head_major(ctx, cq, cache, table, self._gate(proj), heads)
             linear(ctx, heads, self.wo, out, None, epilogue)
             return
         qa = self.absorbed_queries(ctx, cq)
@@ -193,7 +214,7 @@ class LatentAttention(Mixer):
         self.attend(ctx, qa, cache, table, lat)
         heads = ctx.empty((T, self.H * self.dv))
         ops.head_gemm_plain(lat, self.wuv.view(self.H, self.dv, self.rank), heads.view(T, self.H, self.dv),
-                            proj[:, self.off_g:] if self.out_gate else None)
+                            self._gate(proj), gate_heads=self.gate_heads)
         linear(ctx, heads, self.wo, out, None, epilogue)
 
     def forward(self, ctx, h, residual, cache_layer, write_cache=True):

@@ -17,7 +17,7 @@ from ..kernels.ops import EPI_NONE, EPI_BIAS, EPI_RESIDUAL, EPI_SWIGLU
 
 def linear(ctx, x, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
            epilogue: int = EPI_NONE) -> None:
-    """out = epilogue(x @ w.T).
+    """out = epilogue(x @ w.T). With EPI_RESIDUAL a bias, if given, is added as well.
 
     Two products of a layer may share an RMS norm between them without a pass over the rows (bfloat16; many rows: the
     kernels on pairs of SMs; a decode step's few rows: the register-streaming kernel). The product that adds into the residual stream, when the step says which norm reads the
@@ -34,14 +34,14 @@ def linear(ctx, x, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tens
             return
         x = x.normed(ctx)
     norm = ctx.next_norm
-    if (epilogue == EPI_RESIDUAL and bias is None and isinstance(norm, RMSNorm) and norm.weight is not None
+    if (epilogue == EPI_RESIDUAL and isinstance(norm, RMSNorm) and norm.weight is not None
             and out.dtype == torch.float32 and out.shape[1] % 4 == 0 and norm.dim == out.shape[1]):
         if ops.gemm_on_pairs(x, w, out.shape[1], epilogue, ctx.fast):
-            hw, ss = ops.gemm_residual_norm(x, w, out, norm.weight)
+            hw, ss = ops.gemm_residual_norm(x, w, out, norm.weight, bias)
             ctx.memo[("pending norm", id(out))] = PendingNormRows(hw, ss, norm, out)
             return
         if out.shape[1] % 8 == 0 and ops.gemm_skinny_links_norm(x, w, out.shape[1], epilogue, ctx.fast):
-            hw, ss = ops.gemm_skinny_residual_norm(x, w, out, norm.weight)
+            hw, ss = ops.gemm_skinny_residual_norm(x, w, out, norm.weight, bias)
             ctx.memo[("pending norm", id(out))] = PendingNormRows(hw, ss, norm, out)
             return
     ops.gemm(x, w, out, bias, epilogue, fast=ctx.fast)

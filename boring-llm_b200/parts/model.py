@@ -16,10 +16,12 @@ class LayerCall:
     by several entries (its weights run twice), and an entry with `write_cache` false reads the
     cache layer that an earlier entry wrote instead of writing one of its own. A block whose mixer
     keeps several caches (pages AND a state slot: its `cache_spec()` is a tuple) names as many cache
-    layers, as a tuple."""
+    layers, as a tuple. An entry with `enters` true begins a pass of a loop: the model's `reentry` part
+    makes what it reads from the stream and the embedding rows."""
     block: int
     cache: Optional[object]          # int, or a tuple of ints for a block with several caches
     write_cache: bool = True
+    enters: bool = False
 
     def cache_layers(self) -> tuple:
         if self.cache is None:
@@ -36,13 +38,15 @@ class DecoderModel(Part):
 
     def __init__(self, embedding, blocks: Sequence[Part], final_norm, head,
                  schedule: Optional[Sequence[LayerCall]] = None, ignorable_tensors: Sequence[str] = (),
-                 depth_mix: Optional[Sequence[Part]] = None):
-        """`depth_mix`: one part per entry of the run order (`parts.depth.DepthWeightedAverage`); entry i's part turns the
+                 depth_mix: Optional[Sequence[Part]] = None, reentry: Optional[Part] = None):
+        """`reentry`: the part (`parts.depth.StreamReentry`) that runs ahead of every entry of the run order with `enters`.
+        `depth_mix`: one part per entry of the run order (`parts.depth.DepthWeightedAverage`); entry i's part turns the
         streams X_0 .. X_(i+1) (the embedding rows and what each entry so far left) into what the next entry, or the
         final norm, reads. Without it every entry reads what the one before left."""
         super().__init__()
         self.embedding, self.blocks, self.final_norm, self.head = embedding, list(blocks), final_norm, head
         self.depth_mix = list(depth_mix) if depth_mix is not None else None
+        self.reentry = reentry
         self.schedule: List[LayerCall] = list(schedule) if schedule is not None else self._default_order()
         self.keep_streams = None                # a list: every forward pass appends a copy of the stream behind each entry (tests)
         self.ignorable_tensors = tuple(ignorable_tensors)
@@ -57,6 +61,8 @@ class DecoderModel(Part):
                     written.add(c)
                 elif c not in written:
                     raise ValueError(f"an entry reads cache layer {c} before any entry writes it")
+        if any(call.enters for call in self.schedule) and (reentry is None or self.depth_mix is not None):
+            raise ValueError("entries of the run order that begin a pass need a `reentry` part (and no depth mix)")
         if self.depth_mix is not None and len(self.depth_mix) != len(self.schedule):
             raise ValueError(f"{len(self.depth_mix)} depth-mix parts for {len(self.schedule)} entries of the run order")
 
@@ -79,7 +85,8 @@ class DecoderModel(Part):
         return order
 
     def children(self):
-        return (self.embedding, *self.blocks, *(self.depth_mix or ()), self.final_norm, self.head)
+        return (self.embedding, *self.blocks, *(self.depth_mix or ()), *((self.reentry,) if self.reentry is not None else ()),
+                self.final_norm, self.head)
 
     @property
     def vocab_size(self) -> int:
@@ -114,10 +121,15 @@ class DecoderModel(Part):
         if self.depth_mix is not None:
             x = self._forward_depth_mixed(ctx)
             return self._logits(ctx, x)
-        x = self.embedding.forward(ctx)
+        x = x0 = self.embedding.forward(ctx)
+        if self.reentry is not None and not self.schedule[0].enters:
+            x = x0.clone()                      # blocks add into the stream in place; the embedding rows are read again
         for i, call in enumerate(self.schedule):
-            # the norm that reads the stream after this block: the next block's first (the final norm reads a few rows only)
-            after = self.blocks[self.schedule[i + 1].block] if i + 1 < len(self.schedule) else None
+            if call.enters:
+                x = self.reentry.forward(ctx, x, x0)
+            # the norm that reads the stream after this block: the next block's first (the final norm reads a few rows only;
+            # ahead of a pass it is not this stream that the norm reads)
+            after = self.blocks[self.schedule[i + 1].block] if i + 1 < len(self.schedule) and not self.schedule[i + 1].enters else None
             reader = getattr(after, "mixer", None)
             ctx.norm_after_block = getattr(after, "mixer_norm", None) if takes_pending_norm(reader, x.shape[0]) else None
             self.blocks[call.block].forward(ctx, x, call.cache, call.write_cache)

@@ -14,20 +14,23 @@ class RMSNorm(Part):
     """y = x / sqrt(mean(x^2) + eps) * weight, statistics in 32-bit, the weight used as stored
     (src/math.br:18-36). Input: the 32-bit residual stream; output: the engine's activation dtype.
     `scalar_weight`: the checkpoint holds ONE number (a tensor without dimensions) that multiplies every coordinate; it is
-    spread over the width when it is placed, so every kernel that takes an RMS norm's weight takes this one."""
+    spread over the width when it is placed, so every kernel that takes an RMS norm's weight takes this one.
+    `around_zero`: the checkpoint holds w - 1; the weight 1 + w is formed in 32-bit when it is placed."""
 
-    def __init__(self, dim: int, eps: float, names: Dict[str, str], scalar_weight: bool = False):
+    def __init__(self, dim: int, eps: float, names: Dict[str, str], scalar_weight: bool = False, around_zero: bool = False):
         super().__init__(names)
-        self.dim, self.eps, self.scalar_weight = dim, float(eps), bool(scalar_weight)
+        self.dim, self.eps, self.scalar_weight, self.around_zero = dim, float(eps), bool(scalar_weight), bool(around_zero)
         self.weight: Optional[torch.Tensor] = None
 
     def local_specs(self):
-        return {"weight": TensorSpec(() if self.scalar_weight else (self.dim,), NORM)}
+        return {"weight": TensorSpec(() if self.scalar_weight else (self.dim,), BIAS if self.around_zero else NORM)}
 
     def place(self, local, dtype, device):
         w = local["weight"]
         if self.scalar_weight:
             w = w.reshape(1).expand(self.dim).contiguous()
+        if self.around_zero:
+            w = w.to(torch.float32) + 1.0
         self.weight = to_device_vector(w, dtype, device)
 
     def forward(self, ctx, x: torch.Tensor, row_idx: Optional[torch.Tensor] = None, pending_ok: bool = False):
