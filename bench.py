@@ -9,6 +9,7 @@ its roofline.
     python bench.py --design kavotar [--sizes 0.5b|3b] [--layers L]     # the Kavotar design beside Fezopel and Qwen2 at equal sizes
     python bench.py --design miforax [--sizes 0.5b|3b] [--layers L]     # the Miforax design beside Fezopel and Qwen2 at equal sizes
     python bench.py --design dapuzen [--sizes 0.5b|3b] [--layers L]     # the Dapuzen design beside Fezopel and Qwen2 at equal sizes
+    python bench.py --design gipinex [--sizes 0.5b|3b] [--layers L]     # the Gipinex design beside Miforax and Kavotar at equal sizes
 
 One JSON line on standard output. A "step" is one decode step of the whole batch. Requests are real ones: random
 prompts admitted by the scheduler, prefilled in portions through the engine, then decoded; the model comes from the
@@ -460,6 +461,35 @@ def dapuzen_config(sizes, n_layers):
                                       "embedding": {"scale": 1.0}, "layers": layers, "max_position_embeddings": 32768})
 
 
+GIPINEX_PATTERN = ("latent_attention", "attention", "attention")   # repeated over the layers
+GIPINEX_LOOP = 3                                                   # the first three layers run twice
+
+
+def gipinex_config(sizes, n_layers):
+    """A Gipinex model with the width, heads, head size and vocabulary of a Qwen2.5 size and `n_layers` layer RUNS (the first
+    three layers run twice, so three layers less are stored): the attention layers have the Qwen2 heads, the latent layers
+    Miforax's latents; the first layer has the dense feed-forward, the others Miforax's 16 experts of a quarter of its hidden
+    size, 2 a token, beside a shared expert of half of it."""
+    import boring_llm_b200 as b
+    s = SIZES[sizes]
+    d, H, KV, dh, F, V = (s[k] for k in ("hidden_size", "num_attention_heads", "num_key_value_heads", "head_dim",
+                                         "intermediate_size", "vocab_size"))
+    q_rank, kv_rank, rot = MIFORAX_LATENT[sizes]
+    mixers = {
+        "attention": {"heads": H, "kv_heads": KV, "dim": dh, "vdim": dh, "scale": dh ** -0.5},
+        "latent_attention": {"heads": H, "dim": dh, "rot_dim": rot, "vdim": dh, "q_rank": q_rank, "kv_rank": kv_rank,
+                             "scale": (dh + rot) ** -0.5, "rot": {"base": 1000000.0, "dims": rot}},
+    }
+    moe = {"kind": "moe", "expert": {"ff": F // 4 // 8 * 8, "limit": 7.0}, "router": {"experts": MIFORAX_EXPERTS, "top": MIFORAX_TOP},
+           "shared": {"ff": F // 2 // 8 * 8, "limit": 7.0}}
+    loop = min(GIPINEX_LOOP, n_layers // 2)
+    layers = [{"type": GIPINEX_PATTERN[i % len(GIPINEX_PATTERN)], "mixer": mixers[GIPINEX_PATTERN[i % len(GIPINEX_PATTERN)]],
+               "mlp": {"kind": "dense", "ff": F, "limit": 7.0} if i == 0 else moe} for i in range(n_layers - loop)]
+    return b.GipinexConfig.from_dict({"architecture": "Gipinex", "vocab": V, "width": d, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+                                      "loop": {"start": 0, "stop": loop, "times": 2} if loop else None, "layers": layers,
+                                      "max_position_embeddings": 32768})
+
+
 def kernel_time_line(eng, entries, again):
     """The time of every kernel of one step INSIDE its captured graph: the step is captured with a time stamp between
     every two kernels, then `again` (the same shape: it replays that graph) runs, and the stamps of the replay give
@@ -492,7 +522,7 @@ def kernel_time_line(eng, entries, again):
 
 
 def design_bench(args):
-    """Prefill and decode of another design (Fezopel; Kavotar) beside the models it is compared with at equal sizes, random
+    """Prefill and decode of another design beside the models it is compared with at equal sizes, random
     weights, bfloat16: one JSON line."""
     import gc
     import torch
@@ -503,8 +533,8 @@ def design_bench(args):
     pk = peaks()
     n_layers = args.layers or 8
     makers = {"fezopel": fezopel_config, "kavotar": kavotar_config, "miforax": miforax_config, "dapuzen": dapuzen_config,
-              "qwen2": lambda sizes, n: b.Qwen2Config.from_dict({**COMMON, **SIZES[sizes], "num_hidden_layers": n})}
-    names = ("fezopel", "qwen2") if args.design == "fezopel" else (args.design, "fezopel", "qwen2")
+              "gipinex": gipinex_config, "qwen2": lambda sizes, n: b.Qwen2Config.from_dict({**COMMON, **SIZES[sizes], "num_hidden_layers": n})}
+    names = {"fezopel": ("fezopel", "qwen2"), "gipinex": ("gipinex", "miforax", "kavotar")}.get(args.design, (args.design, "fezopel", "qwen2"))
     out = {"design": args.design, "beside": list(names[1:]), "sizes": args.sizes, "layers": n_layers, "dtype": "bf16", "data": "synthetic",
            "context": CONTEXT, "prefill_tokens": PREFILL_TOKENS, "peaks": pk["source"], "models": {}}
     if args.design == "fezopel":
@@ -514,6 +544,9 @@ def design_bench(args):
     elif args.design == "dapuzen":
         out.update(pattern=list(DAPUZEN_PATTERN), window=DAPUZEN_WINDOW, state=DAPUZEN_STATE,
                    experts=[DAPUZEN_EXPERTS, DAPUZEN_TOP, DAPUZEN_IDENTITY, DAPUZEN_GROUPS, DAPUZEN_KEEP])
+    elif args.design == "gipinex":
+        out.update(pattern=list(GIPINEX_PATTERN), loop=[0, GIPINEX_LOOP, 2], experts=[MIFORAX_EXPERTS, MIFORAX_TOP],
+                   latent=list(MIFORAX_LATENT[args.sizes]))
     else:
         out.update(pattern=list(KAVOTAR_PATTERN), chunk=KAVOTAR_CHUNK, experts=[KAVOTAR_EXPERTS, KAVOTAR_TOP, KAVOTAR_GROUPS, KAVOTAR_KEEP])
     clocks = ClockSampler()
@@ -579,8 +612,8 @@ def main():
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "prefill4", "mixed"],
                     help="run one part only and print its figures (for profilers; not the benchmark line)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--design", default="", choices=["", "fezopel", "kavotar", "miforax", "dapuzen"],
-                    help="measure another design beside Qwen2 at equal sizes instead of the default workload (its own JSON line)")
+    ap.add_argument("--design", default="", choices=["", "fezopel", "kavotar", "miforax", "dapuzen", "gipinex"],
+                    help="measure another design beside its closest models at equal sizes instead of the default workload (its own JSON line)")
     args = ap.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":
