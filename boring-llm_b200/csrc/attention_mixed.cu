@@ -32,8 +32,9 @@ constexpr int PAD = 8;                // bfloat16 elements of padding per shared
 constexpr int MAX_DH = 512;           // the plain kernel's head size
 constexpr int PLAIN_WARPS = 4;
 constexpr int PREP_THREADS = 128;
-constexpr int PREP_HEADS = 4;         // heads whose mixed queries one block of bl_mixed_prep makes
+constexpr int PREP_FEW_ROWS = 256;    // up to so many tokens a block of bl_mixed_prep makes the mixed queries of four heads, with more of all
 constexpr int STAGES = 3;             // prefill ring
+constexpr int MAX_DECODE_WARPS = 8;   // warps of a decode block
 constexpr int MAX_CLUSTER = 16;       // slices merged through distributed shared memory
 
 // ---- norms, mixed queries, keys into the pages ----------------------------------------------------------------------------
@@ -41,14 +42,17 @@ template <typename TT>
 __global__ void __launch_bounds__(PREP_THREADS)
 mixed_prep_kernel(const float* proj, int ld, int off_k, const float* __restrict__ talk, float eps, const int* __restrict__ positions,
                   const int* __restrict__ tok_req, const int* __restrict__ block_table, int max_pages, TT* __restrict__ q_out,
-                  TT* __restrict__ k_cache, float* __restrict__ k_rms, int rms_stride, int H, int KV, int dh, int page_size) {
+                  TT* __restrict__ k_cache, float* __restrict__ k_rms, int rms_stride, int H, int KV, int dh, int page_size, int heads_per_block) {
     bl_pdl_trigger();
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     float* qn = sm;                                    // [H * dh] the token's normed queries
-    float* coef = qn + H * dh;                         // [PREP_HEADS][H] this block's rows of the mix
-    const int t = blockIdx.x, h0 = blockIdx.y * PREP_HEADS, nh = min(PREP_HEADS, H - h0);
+    float* coef = qn + ((H * dh + 3) & ~3);            // this block's rows of the mix, four heads side by side: [heads / 4][H][4]
+    const int t = blockIdx.x, h0 = blockIdx.y * heads_per_block, nh = min(heads_per_block, H - h0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int i = threadIdx.x; i < PREP_HEADS * H; i += PREP_THREADS) coef[i] = i / H < nh ? talk[(size_t)(h0 + i / H) * H + i % H] : 0.f;
+    for (int i = threadIdx.x; i < ((nh + 3) & ~3) * H; i += PREP_THREADS) {
+        const int hh = (i / (4 * H)) * 4 + (i & 3), g = (i >> 2) % H;
+        coef[i] = hh < nh ? talk[(size_t)(h0 + hh) * H + g] : 0.f;
+    }
     bl_pdl_wait();
     const float* row = proj + (size_t)t * ld;
     for (int g = warp; g < H; g += PREP_THREADS / 32) {
@@ -74,16 +78,23 @@ mixed_prep_kernel(const float* proj, int ld, int off_k, const float* __restrict_
     __syncthreads();
     const int G = H / KV;
     for (int e = threadIdx.x; e < KV * dh; e += PREP_THREADS) {
-        const int c = e / dh, d = e % dh;
-        float acc[PREP_HEADS];
-#pragma unroll
-        for (int i = 0; i < PREP_HEADS; ++i) acc[i] = 0.f;
-        for (int g = c * G; g < (c + 1) * G; ++g) {
-            const float v = qn[g * dh + d];
-#pragma unroll
-            for (int i = 0; i < PREP_HEADS; ++i) acc[i] = fmaf(coef[i * H + g], v, acc[i]);
+        const int c = e / dh, d = e - c * dh;
+        for (int i0 = 0; i0 < nh; i0 += 4) {
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4* cf = reinterpret_cast<const float4*>(coef + (i0 * H + c * G * 4));
+            const float* qg = qn + c * G * dh + d;
+            for (int g = 0; g < G; ++g) {
+                const float v = qg[g * dh];
+                const float4 w = cf[g];
+                acc.x = fmaf(w.x, v, acc.x); acc.y = fmaf(w.y, v, acc.y); acc.z = fmaf(w.z, v, acc.z); acc.w = fmaf(w.w, v, acc.w);
+            }
+            TT* dst = q_out + ((size_t)t * H + h0 + i0) * KV * dh + e;
+            const size_t next = (size_t)KV * dh;
+            bl_store(dst, acc.x);
+            if (i0 + 1 < nh) bl_store(dst + next, acc.y);
+            if (i0 + 2 < nh) bl_store(dst + 2 * next, acc.z);
+            if (i0 + 3 < nh) bl_store(dst + 3 * next, acc.w);
         }
-        for (int i = 0; i < nh; ++i) bl_store(q_out + ((size_t)t * H + h0 + i) * KV * dh + e, acc[i]);
     }
 }
 
@@ -210,6 +221,33 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
+// Two neighbouring scores at a time: Blackwell's packed 32-bit operations (each half rounded as its scalar form).
+__device__ __forceinline__ unsigned long long pack2(float lo, float hi) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(unsigned long long v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
 // The running maximum and sum of two rows (g and g + 8 of a warp's 16) take in NT tiles of 8 keys whose raw scores are s;
 // afterwards s holds the weights 2^(score - m). Key n * 8 + 2t + e of the tiles is key `key0` + that.
 template <int NT, int NO>
@@ -217,26 +255,26 @@ __device__ __forceinline__ void softmax_step(float (&s)[NT][4], float (&o)[NO][4
                                              const float (&slope)[2], int key0, float scale_log2) {
     const int t = threadIdx.x & 3;
     const bool all_seen = key0 + NT * 8 - 1 <= min(pos[0], pos[1]);
-    float mx[2] = {-INFINITY, -INFINITY};
+    const unsigned long long sc2 = pack2(scale_log2, scale_log2);
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         const float b0 = -slope[h] * (float)(pos[h] - key0 - 2 * t);       // the bias of this lane's first key; a key on adds a slope
+        const unsigned long long first2 = pack2(b0, b0), slope2 = pack2(slope[h], slope[h]);
+        float mx = -INFINITY;
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                float v = fmaf(s[n][2 * h + e], scale_log2, fmaf(slope[h], (float)(n * 8 + e), b0));
-                if (!all_seen && key0 + n * 8 + 2 * t + e > pos[h]) v = -INFINITY;
-                s[n][2 * h + e] = v;
-                mx[h] = fmaxf(mx[h], v);
+            const unsigned long long bias2 = fma2(slope2, pack2((float)(n * 8), (float)(n * 8 + 1)), first2);
+            float2 v = unpack2(fma2(pack2(s[n][2 * h], s[n][2 * h + 1]), sc2, bias2));
+            if (!all_seen) {
+                if (key0 + n * 8 + 2 * t > pos[h]) v.x = -INFINITY;
+                if (key0 + n * 8 + 2 * t + 1 > pos[h]) v.y = -INFINITY;
             }
+            s[n][2 * h] = v.x; s[n][2 * h + 1] = v.y;
+            mx = fmaxf(mx, fmaxf(v.x, v.y));
         }
-    }
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-        const float m_new = fmaxf(m[h], mx[h]);
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float m_new = fmaxf(m[h], mx);
         const float m_use = m_new == -INFINITY ? 0.f : m_new;              // a row that has seen no key yet
         if (m_new != m[h]) {
             const float alpha = ex2(m[h] - m_use);                         // 2^-inf = 0 on the first block
@@ -245,16 +283,22 @@ __device__ __forceinline__ void softmax_step(float (&s)[NT][4], float (&o)[NO][4
 #pragma unroll
             for (int n = 0; n < NO; ++n) { o[n][2 * h] *= alpha; o[n][2 * h + 1] *= alpha; }
         }
+        const unsigned long long less2 = pack2(-m_use, -m_use);
+        unsigned long long sum2 = pack2(0.f, 0.f);
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const float p = ex2(s[n][2 * h + e] - m_use);
-                s[n][2 * h + e] = p;
-                l[h] += p;
-            }
+            const float2 d = unpack2(add2(pack2(s[n][2 * h], s[n][2 * h + 1]), less2));
+            s[n][2 * h] = ex2(d.x); s[n][2 * h + 1] = ex2(d.y);
+            sum2 = add2(sum2, pack2(s[n][2 * h], s[n][2 * h + 1]));
         }
+        const float2 sum = unpack2(sum2);
+        l[h] += sum.x + sum.y;
     }
+}
+// The weights of two keys times the keys' root mean squares, as the left operand's word.
+__device__ __forceinline__ unsigned weigh(float p0, float p1, unsigned long long rms2) {
+    const float2 v = unpack2(mul2(pack2(p0, p1), rms2));
+    return pack_bf16(v.x, v.y);
 }
 
 // ND: head size in chunks of 16 values (rounded up; the columns past dh are zeros in shared memory).
@@ -274,31 +318,41 @@ struct Sizes {
 };
 
 // Keys [key0, key0 + 64) of key/value head c into a stage; with `rms` also their root mean squares. Keys past hi become
-// zeros: they are masked anyway, and zeros keep the products finite whatever an earlier request left in a page.
+// zeros: they are masked anyway, and zeros keep the products finite whatever an earlier request left in a page. Eight threads
+// copy a row; the four rows of a thread are the same row of the block's four pages (asked for a tile ahead: `pages`).
 template <int ND>
-__device__ __forceinline__ void load_tile(__nv_bfloat16* ks, float* rms, const MixedParams& p, const int* table, int c, int key0, int hi) {
+__device__ __forceinline__ void load_tile(__nv_bfloat16* ks, float* rms, const MixedParams& p, const int (&pages)[KB / PAGE], int c, int key0, int hi) {
     constexpr int ROW = Sizes<ND>::ROW;
-    const int ch = p.dh / 8, c0 = threadIdx.x & 7;
+    const int row = threadIdx.x >> 3, c0 = threadIdx.x & 7, ch = p.dh / 8;
+    const size_t in_page = (size_t)(c * PAGE + row) * p.dh + c0 * 8, page_size = (size_t)p.KV * PAGE * p.dh;
+    __nv_bfloat16* dst = ks + row * ROW + c0 * 8;
+    const bool whole = key0 + KB - 1 <= hi;
 #pragma unroll
-    for (int r = threadIdx.x >> 3; r < KB; r += 16) {                      // eight threads a row
-        const int key = key0 + r;
-        __nv_bfloat16* dst = ks + r * ROW;
-        if (key <= hi) {
-            const __nv_bfloat16* src = p.kc + (((size_t)table[key / PAGE] * p.KV + c) * PAGE + key % PAGE) * p.dh;
-            for (int i = c0; i < ch; i += 8) cp_async16(dst + i * 8, src + i * 8);
+    for (int q = 0; q < KB / PAGE; ++q) {
+        __nv_bfloat16* d = dst + q * PAGE * ROW;
+        if (whole || key0 + q * PAGE + row <= hi) {
+            const __nv_bfloat16* src = p.kc + (size_t)pages[q] * page_size + in_page;
+#pragma unroll
+            for (int x = 0; x < (ND + 3) / 4; ++x) if (c0 + 8 * x < ch) cp_async16(d + 64 * x, src + 64 * x);
         } else {
-            for (int i = c0; i < ch; i += 8) *reinterpret_cast<uint4*>(dst + i * 8) = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+            for (int x = 0; x < (ND + 3) / 4; ++x) if (c0 + 8 * x < ch) *reinterpret_cast<uint4*>(d + 64 * x) = make_uint4(0u, 0u, 0u, 0u);
         }
     }
     if (rms && threadIdx.x < KB) {
-        const int key = key0 + threadIdx.x;
-        if (key <= hi) cp_async4(rms + threadIdx.x, p.k_rms + ((size_t)table[key / PAGE] * p.KV + c) * PAGE + key % PAGE);
+        if (whole || key0 + (int)threadIdx.x <= hi)
+        {
+            const int lo_page = (threadIdx.x & 16) ? pages[1] : pages[0], hi_page = (threadIdx.x & 16) ? pages[3] : pages[2];
+            cp_async4(rms + threadIdx.x, p.k_rms + ((size_t)((threadIdx.x & 32) ? hi_page : lo_page) * p.KV + c) * PAGE + threadIdx.x % PAGE);
+        }
         else rms[threadIdx.x] = 0.f;
     }
 }
 
+template <int ND> constexpr int PREFILL_BLOCKS = ND <= 6 ? 3 : 2;          // prefill blocks an SM holds, by registers
+
 template <int ND>
-__global__ void __launch_bounds__(128, ND <= 4 ? 3 : 2)
+__global__ void __launch_bounds__(128, PREFILL_BLOCKS<ND>)
 attention_mixed_prefill_kernel(const MixedParams p) {
     constexpr int ROW = Sizes<ND>::ROW, TILE = Sizes<ND>::TILE, DP = Sizes<ND>::DP;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -308,7 +362,8 @@ attention_mixed_prefill_kernel(const MixedParams p) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int mi = lane >> 3, ri = lane & 7;                               // ldmatrix: which 8x8 matrix, which row of it
     bl_pdl_trigger();
-    const int unit = gridDim.x / p.H - 1 - blockIdx.x / p.H;               // late tiles see the most keys: they go first
+    // late tiles of a request see the most keys: they go first, the short ones fill the tail
+    const int unit = gridDim.x / p.H - 1 - blockIdx.x / p.H;
     const int r = p.work[2 * unit], tok0 = p.work[2 * unit + 1];
     const int head = blockIdx.x % p.H, own = head / (p.H / p.KV);
     const int q_begin = p.cu_q[r], q_len = p.cu_q[r + 1] - q_begin, ctx = p.ctx_len[r];
@@ -341,66 +396,82 @@ attention_mixed_prefill_kernel(const MixedParams p) {
             else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
         }
     }
-    // tile i: keys of block i / KV, of the key/value head `own` last
-    auto issue = [&](int i) {
-        const int ci = i % p.KV, c = (own + 1 + ci) % p.KV, st = i % STAGES;
-        load_tile<ND>(ks + st * TILE, ci == p.KV - 1 ? rs + st * KB : nullptr, p, table, c, (i / p.KV) * KB, hi);
+    // the tiles in their order: key block by key block, the key/value heads in a ring that ends with `own`
+    const int c_begin = own + 1 == p.KV ? 0 : own + 1;
+    int left = n_tiles, i_key = 0, i_c = c_begin, i_st = 0;                // the next tile to ask for
+    int pages[KB / PAGE];                                                  // ... and its pages
+    auto find_pages = [&]() {
+#pragma unroll
+        for (int q = 0; q < KB / PAGE; ++q) pages[q] = i_key + q * PAGE <= hi ? table[i_key / PAGE + q] : 0;
+    };
+    find_pages();
+    auto issue = [&]() {
+        if (left > 0) {
+            load_tile<ND>(ks + i_st * TILE, i_c == own ? rs + i_st * KB : nullptr, p, pages, i_c, i_key, hi);
+            if (i_c == own) { i_key += KB; find_pages(); }
+            if (++i_c == p.KV) i_c = 0;
+            if (++i_st == STAGES) i_st = 0;
+            --left;
+        }
+        cp_async_commit();
     };
 #pragma unroll
-    for (int i = 0; i < STAGES - 1; ++i) {                                 // (the queries belong to the first group)
-        if (i < n_tiles) issue(i);
-        cp_async_commit();
-    }
+    for (int i = 0; i < STAGES - 1; ++i) issue();                          // (the queries belong to the first group)
     float o[2 * ND][4];
 #pragma unroll
     for (int n = 0; n < 2 * ND; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     float s[KB / 8][4];
-    int ci = 0, st = 0;
+#pragma unroll
+    for (int n = 0; n < KB / 8; ++n) { s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f; }
+    int c = c_begin, st = 0, key0 = 0;
+    const __nv_bfloat16* q_row = qs + (warp * 16 + (mi & 1) * 8 + ri) * ROW + (mi >> 1) * 8;
+    const __nv_bfloat16* k_row = ks + ((mi >> 1) * 8 + ri) * ROW + (mi & 1) * 8;
+    const __nv_bfloat16* v_row = ks + ((mi & 1) * 8 + ri) * ROW + (mi >> 1) * 8;
     for (int i = 0; i < n_tiles; ++i) {
         cp_async_wait<STAGES - 2>();
         __syncthreads();                                                   // tile i has landed; everybody is through with tile i - 1
-        if (i + STAGES - 1 < n_tiles) issue(i + STAGES - 1);
-        cp_async_commit();
-        const __nv_bfloat16* kt = ks + st * TILE;
-        const __nv_bfloat16* qt = qs + ((own + 1 + ci) % p.KV) * TILE + warp * 16 * ROW;
-        if (ci == 0) {
-#pragma unroll
-            for (int n = 0; n < KB / 8; ++n) { s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f; }
-        }
+        issue();
+        const __nv_bfloat16* kt = k_row + st * TILE;
+        const __nv_bfloat16* qt = q_row + c * TILE;
 #pragma unroll
         for (int kk = 0; kk < ND; ++kk) {
             unsigned a[4];
-            ldmatrix_x4(a, qt + ((mi & 1) * 8 + ri) * ROW + kk * 16 + (mi >> 1) * 8);
+            ldmatrix_x4(a, qt + kk * 16);
 #pragma unroll
             for (int np = 0; np < KB / 16; ++np) {
                 unsigned b[4];
-                ldmatrix_x4(b, kt + (np * 16 + (mi >> 1) * 8 + ri) * ROW + kk * 16 + (mi & 1) * 8);
+                ldmatrix_x4(b, kt + np * 16 * ROW + kk * 16);
                 mma_bf16(s[2 * np], a, b[0], b[1]);
                 mma_bf16(s[2 * np + 1], a, b[2], b[3]);
             }
         }
-        if (ci == p.KV - 1) {                                              // the block's scores are complete, its values are this tile
-            softmax_step<KB / 8, 2 * ND>(s, o, m, l, pos, slope, (i / p.KV) * KB, p.scale_log2);
-            const float* rt = rs + st * KB;
+        if (c == own) {                                                    // the block's scores are complete, its values are this tile
+            softmax_step<KB / 8, 2 * ND>(s, o, m, l, pos, slope, key0, p.scale_log2);
+            const float* rt = rs + st * KB + 2 * t;
+            const __nv_bfloat16* vt = v_row + st * TILE;
 #pragma unroll
             for (int kk = 0; kk < KB / 16; ++kk) {
-                const float2 r0 = *reinterpret_cast<const float2*>(rt + kk * 16 + 2 * t), r1 = *reinterpret_cast<const float2*>(rt + kk * 16 + 8 + 2 * t);
+                const unsigned long long r0 = *reinterpret_cast<const unsigned long long*>(rt + kk * 16);
+                const unsigned long long r1 = *reinterpret_cast<const unsigned long long*>(rt + kk * 16 + 8);
                 unsigned a[4];
-                a[0] = pack_bf16(s[2 * kk][0] * r0.x, s[2 * kk][1] * r0.y);
-                a[1] = pack_bf16(s[2 * kk][2] * r0.x, s[2 * kk][3] * r0.y);
-                a[2] = pack_bf16(s[2 * kk + 1][0] * r1.x, s[2 * kk + 1][1] * r1.y);
-                a[3] = pack_bf16(s[2 * kk + 1][2] * r1.x, s[2 * kk + 1][3] * r1.y);
+                a[0] = weigh(s[2 * kk][0], s[2 * kk][1], r0);
+                a[1] = weigh(s[2 * kk][2], s[2 * kk][3], r0);
+                a[2] = weigh(s[2 * kk + 1][0], s[2 * kk + 1][1], r1);
+                a[3] = weigh(s[2 * kk + 1][2], s[2 * kk + 1][3], r1);
 #pragma unroll
                 for (int np = 0; np < ND; ++np) {
                     unsigned b[4];
-                    ldmatrix_x4_trans(b, kt + (kk * 16 + (mi & 1) * 8 + ri) * ROW + np * 16 + (mi >> 1) * 8);
+                    ldmatrix_x4_trans(b, vt + kk * 16 * ROW + np * 16);
                     mma_bf16(o[2 * np], a, b[0], b[1]);
                     mma_bf16(o[2 * np + 1], a, b[2], b[3]);
                 }
             }
+            key0 += KB;
+#pragma unroll
+            for (int n = 0; n < KB / 8; ++n) { s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f; }
         }
-        if (++ci == p.KV) ci = 0;
+        if (++c == p.KV) c = 0;
         if (++st == STAGES) st = 0;
     }
     cp_async_wait<0>();
@@ -445,31 +516,43 @@ __device__ __forceinline__ float2 ld_cluster_f2(uint32_t a) {
     return v;
 }
 
-// One warp copies the page that holds keys [key0, key0 + 16), of every key/value head, into a stage of its own.
+// One warp copies the page that holds keys [key0, key0 + 16), of every key/value head, into a stage of its own. Eight lanes
+// copy a row; all rows of a page lie together.
 template <int ND>
 __device__ __forceinline__ void load_page(__nv_bfloat16* ks, float* rms, const MixedParams& p, const int* table, int key0, int hi) {
     constexpr int ROW = Sizes<ND>::ROW;
-    const int lane = threadIdx.x & 31, ch = p.dh / 8;
+    const int lane = threadIdx.x & 31, ch = p.dh / 8, c0 = lane & 7;
     const int live = min(PAGE, hi - key0 + 1);                             // keys of the page that exist (may be <= 0)
     const size_t page = live > 0 ? (size_t)table[key0 / PAGE] : 0;
-    const __nv_bfloat16* src = p.kc + page * p.KV * PAGE * p.dh;
-    const int c0 = lane & 7;                                               // eight lanes a row: no division by ch
-    for (int rr = lane >> 3; rr < p.KV * PAGE; rr += 4) {
-        __nv_bfloat16* dst = ks + rr * ROW;
-        if (rr % PAGE < live) {
-            for (int x = c0; x < ch; x += 8) cp_async16(dst + x * 8, src + (size_t)rr * p.dh + x * 8);
-        } else {
-            for (int x = c0; x < ch; x += 8) *reinterpret_cast<uint4*>(dst + x * 8) = make_uint4(0u, 0u, 0u, 0u);
+    const int rows = p.KV * PAGE, step = 4 * p.dh;
+    const __nv_bfloat16* src = p.kc + (page * rows + (lane >> 3)) * p.dh + c0 * 8;
+    __nv_bfloat16* dst = ks + (lane >> 3) * ROW + c0 * 8;
+    const float* rsrc = p.k_rms + page * rows;
+    if (live == PAGE) {
+#pragma unroll 4
+        for (int rr = 0; rr < rows; rr += 4, src += step, dst += 4 * ROW) {
+#pragma unroll
+            for (int x = 0; x < (ND + 3) / 4; ++x) if (c0 + 8 * x < ch) cp_async16(dst + 64 * x, src + 64 * x);
+        }
+        for (int rr = lane * 4; rr < rows; rr += 128) cp_async16(rms + rr, rsrc + rr);
+        return;
+    }
+    for (int rr = lane >> 3; rr < rows; rr += 4, src += step, dst += 4 * ROW) {
+#pragma unroll
+        for (int x = 0; x < (ND + 3) / 4; ++x) {
+            if (c0 + 8 * x >= ch) continue;
+            if (rr % PAGE < live) cp_async16(dst + 64 * x, src + 64 * x);
+            else *reinterpret_cast<uint4*>(dst + 64 * x) = make_uint4(0u, 0u, 0u, 0u);
         }
     }
-    for (int rr = lane; rr < p.KV * PAGE; rr += 32) {
-        if (rr % PAGE < live) cp_async4(rms + rr, p.k_rms + page * p.KV * PAGE + rr);
+    for (int rr = lane; rr < rows; rr += 32) {
+        if (rr % PAGE < live) cp_async4(rms + rr, rsrc + rr);
         else rms[rr] = 0.f;
     }
 }
 
 template <int ND, int WSTAGES>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(MAX_DECODE_WARPS * 32, ND <= 4 ? 2 : 1)
 attention_mixed_decode_kernel(const MixedParams p) {
     constexpr int ROW = Sizes<ND>::ROW, DP = Sizes<ND>::DP;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -538,35 +621,45 @@ attention_mixed_decode_kernel(const MixedParams p) {
 #pragma unroll
     for (int n = 0; n < 2 * ND; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    const __nv_bfloat16* q_row = qs + ((mi & 1) * 8 + ri) * ROW + (mi >> 1) * 8;
+    const __nv_bfloat16* k_row = stage_keys(0) + ((mi >> 1) * 8 + ri) * ROW + (mi & 1) * 8;
+    const __nv_bfloat16* v_row = stage_keys(0) + ((mi & 1) * 8 + ri) * ROW + (mi >> 1) * 8;
     for (int i = 0; i < nb; ++i) {
         const int pending = issued - (i + 1);
         if (pending >= 2) cp_async_wait<2>(); else if (pending == 1) cp_async_wait<1>(); else cp_async_wait<0>();
         __syncwarp();
-        const __nv_bfloat16* kt = stage_keys(i % WSTAGES);
         const float* rt = stage_rms(i % WSTAGES);
-        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        for (int c = 0; c < p.KV; ++c) {
+        // two sets of sums (even and odd chunks of the head size), so that a product does not wait for the one before it
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}}, s2[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        const __nv_bfloat16* qt = q_row;
+        const __nv_bfloat16* kt = k_row + (size_t)(i % WSTAGES) * (stage_bytes / 2);
+#pragma unroll 2
+        for (int c = 0; c < p.KV; ++c, qt += 16 * ROW, kt += PAGE * ROW) {
 #pragma unroll
             for (int kk = 0; kk < ND; ++kk) {
                 unsigned a[4], b[4];
-                ldmatrix_x4(a, qs + (c * 16 + (mi & 1) * 8 + ri) * ROW + kk * 16 + (mi >> 1) * 8);
-                ldmatrix_x4(b, kt + (c * PAGE + (mi >> 1) * 8 + ri) * ROW + kk * 16 + (mi & 1) * 8);
-                mma_bf16(s[0], a, b[0], b[1]);
-                mma_bf16(s[1], a, b[2], b[3]);
+                ldmatrix_x4(a, qt + kk * 16);
+                ldmatrix_x4(b, kt + kk * 16);
+                mma_bf16(kk & 1 ? s2[0] : s[0], a, b[0], b[1]);
+                mma_bf16(kk & 1 ? s2[1] : s[1], a, b[2], b[3]);
             }
         }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { s[0][e] += s2[0][e]; s[1][e] += s2[1][e]; }
         softmax_step<2, 2 * ND>(s, o, m, l, pos, slope, key_of(i), p.scale_log2);
+        const __nv_bfloat16* vt = v_row + (size_t)(i % WSTAGES) * (stage_bytes / 2);
         for (int c = c_first; c <= c_last; ++c) {
-            const float2 r0 = *reinterpret_cast<const float2*>(rt + c * PAGE + 2 * t), r1 = *reinterpret_cast<const float2*>(rt + c * PAGE + 8 + 2 * t);
+            const unsigned long long r0 = *reinterpret_cast<const unsigned long long*>(rt + c * PAGE + 2 * t);
+            const unsigned long long r1 = *reinterpret_cast<const unsigned long long*>(rt + c * PAGE + 8 + 2 * t);
             unsigned a[4];
-            a[0] = kv0 == c ? pack_bf16(s[0][0] * r0.x, s[0][1] * r0.y) : 0u;
-            a[1] = kv1 == c ? pack_bf16(s[0][2] * r0.x, s[0][3] * r0.y) : 0u;
-            a[2] = kv0 == c ? pack_bf16(s[1][0] * r1.x, s[1][1] * r1.y) : 0u;
-            a[3] = kv1 == c ? pack_bf16(s[1][2] * r1.x, s[1][3] * r1.y) : 0u;
+            a[0] = kv0 == c ? weigh(s[0][0], s[0][1], r0) : 0u;
+            a[1] = kv1 == c ? weigh(s[0][2], s[0][3], r0) : 0u;
+            a[2] = kv0 == c ? weigh(s[1][0], s[1][1], r1) : 0u;
+            a[3] = kv1 == c ? weigh(s[1][2], s[1][3], r1) : 0u;
 #pragma unroll
             for (int np = 0; np < ND; ++np) {
                 unsigned b[4];
-                ldmatrix_x4_trans(b, kt + (c * PAGE + (mi & 1) * 8 + ri) * ROW + np * 16 + (mi >> 1) * 8);
+                ldmatrix_x4_trans(b, vt + c * PAGE * ROW + np * 16);
                 mma_bf16(o[2 * np], a, b[0], b[1]);
                 mma_bf16(o[2 * np + 1], a, b[2], b[3]);
             }
@@ -672,8 +765,9 @@ constexpr int SMEM_LIMIT = 227 * 1024;
 
 template <int ND>
 bool decode_shape(int KV, int* warps, int* stages) {
-    // four warps with three stages each, or what fits: two blocks an SM where that leaves three stages
-    const int shapes[5][2] = {{4, 3}, {4, 2}, {2, 3}, {2, 2}, {1, 2}};
+    // eight warps with three stages each where two such blocks fit an SM, else what fits
+    if (Sizes<ND>::decode_bytes(KV, 8, 3) <= SMEM_LIMIT / 2) { *warps = 8; *stages = 3; return true; }
+    const int shapes[6][2] = {{8, 2}, {4, 3}, {4, 2}, {2, 3}, {2, 2}, {1, 2}};
     for (const auto& s : shapes)
         if (Sizes<ND>::decode_bytes(KV, s[0], s[1]) <= SMEM_LIMIT) { *warps = s[0]; *stages = s[1]; return true; }
     return false;
@@ -681,7 +775,11 @@ bool decode_shape(int KV, int* warps, int* stages) {
 
 template <int ND>
 int launch_prefill(const MixedParams& p, int n_tiles, cudaStream_t s) {
-    const int bytes = Sizes<ND>::prefill_bytes(p.KV);
+    // A launch whose blocks are all resident at once cannot even out its long and short blocks. So a launch of few blocks asks for
+    // more shared memory than it uses, which leaves two blocks an SM, and the rest start as places become free (2,048 tokens, 14
+    // heads of 64 values: 81 us with two blocks an SM, 101 with three, 110 with four; 4,096 tokens want three).
+    int bytes = Sizes<ND>::prefill_bytes(p.KV);
+    if ((long long)n_tiles * p.H * 2 < 148LL * 3 * PREFILL_BLOCKS<ND> && bytes < SMEM_LIMIT / 3) bytes = SMEM_LIMIT / 3;
     static thread_local int allowed = 0;
     if (bytes > allowed) {
         BL_CUDA(cudaFuncSetAttribute(attention_mixed_prefill_kernel<ND>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
@@ -732,8 +830,9 @@ int decode_resident(int KV) {
     int dev = 0, sms = 0;
     if (cudaGetDevice(&dev) != cudaSuccess) return 0;
     if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return 0;
-    const int per_sm = SMEM_LIMIT / (bytes + 1024);
-    return sms * (per_sm < 1 ? 1 : (per_sm > 4 ? 4 : per_sm));
+    const int by_smem = SMEM_LIMIT / (bytes + 1024), by_regs = (ND <= 4 ? 16 : 8) / warps;
+    const int per_sm = by_smem < by_regs ? by_smem : by_regs;
+    return sms * (per_sm < 1 ? 1 : per_sm);
 }
 
 int check(const char* who, const MixedParams& p, int page_size) {
@@ -765,14 +864,15 @@ extern "C" int bl_mixed_prep(const float* proj, int ld, int off_k, const float* 
     if (H <= 0 || KV <= 0 || H % KV != 0 || dh <= 0) BL_FAIL("bl_mixed_prep: %d heads of %d values on %d key/value heads", H, dh, KV);
     if (off_k < H * dh || off_k + KV * dh > ld || page_size <= 0 || max_pages <= 0) BL_FAIL("bl_mixed_prep: keys from column %d do not fit rows of %d", off_k, ld);
     if (k_cache && (!k_rms || rms_stride <= 0)) BL_FAIL("bl_mixed_prep: keys without a place for their root mean squares");
-    const size_t smem = (size_t)(H * dh + PREP_HEADS * H) * sizeof(float);
+    const int per_block = T <= PREP_FEW_ROWS ? 4 : (H + 3) & ~3;
+    const size_t smem = (size_t)(((H * dh + 3) & ~3) + per_block * H) * sizeof(float);
     if (smem > 160 * 1024) BL_FAIL("bl_mixed_prep: %d heads of %d values are too many for shared memory", H, dh);
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid(T, (H + PREP_HEADS - 1) / PREP_HEADS);
+    const dim3 grid(T, (H + per_block - 1) / per_block);
 #define BL_GO(TT) do { \
         if (smem > 48 * 1024) BL_CUDA(cudaFuncSetAttribute(mixed_prep_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         BL_CUDA(bl_launch_dependent(mixed_prep_kernel<TT>, grid, dim3(PREP_THREADS), smem, s, proj, ld, off_k, talk, eps, positions, tok_req, \
-                                    block_table, max_pages, (TT*)q_out, (TT*)k_cache, k_rms, rms_stride, H, KV, dh, page_size)); } while (0)
+                                    block_table, max_pages, (TT*)q_out, (TT*)k_cache, k_rms, rms_stride, H, KV, dh, page_size, per_block)); } while (0)
     if (dtype == BL_F32) BL_GO(float);
     else if (dtype == BL_BF16) BL_GO(__nv_bfloat16);
     else BL_FAIL("bl_mixed_prep: unknown dtype %d", dtype);
