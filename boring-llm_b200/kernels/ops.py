@@ -1690,3 +1690,80 @@ def attention_mixed_splits(n: int, H: int, KV: int, dh: int, longest: int) -> in
     units = max(1, n * (-(-H // 16)))
     most = MIXED_MAX_SPLITS if units * MIXED_MAX_SPLITS <= _sms() // 2 else MIXED_MAX_SPLITS // 2
     return max(1, min(-(-longest // 64), _mixed_resident[key] // units, most))
+
+
+def rope_decay_prep(proj: torch.Tensor, off_k: int, positions: torch.Tensor, inv_freq: torch.Tensor, rot_half: int,
+                    head_decay: torch.Tensor, k_scale: float, H: int, dk: int):
+    """In front of a recurrence with a fixed decay per head: (q, k, decay), each 32-bit [T, H * dk], from the joined
+    projections (q first, k from column off_k): q and k rotated by position (pairs (i, i + rot_half) of each head's first
+    2 * rot_half values, 32-bit angles), k times k_scale, decay[t, h, :] = head_decay[h]."""
+    T = proj.shape[0]
+    ld = _rows32(proj, "proj", T, off_k + H * dk)
+    _need(positions, "positions", torch.int32, (T,)); _need(inv_freq, "inv_freq", torch.float32); _need(head_decay, "head_decay", torch.float32, (H,))
+    if inv_freq.numel() < rot_half:
+        raise KernelError("inv_freq: fewer entries than rotated pairs")
+    q, k, decay = (torch.empty((T, H * dk), dtype=torch.float32, device=proj.device) for _ in range(3))
+    _call(_lib().bl_rope_decay_prep, _p(proj), ld, off_k, _p(positions), _p(inv_freq), rot_half, _p(head_decay), ctypes.c_float(k_scale),
+          _p(q), _p(k), _p(decay), T, H, dk, _stream())
+    return q, k, decay
+
+
+def ssd_prep(raw: torch.Tensor, dt_bias: torch.Tensor, rate: torch.Tensor, x: torch.Tensor, H: int, n_state: int, dv: int):
+    """In front of a selective state-space recurrence: dt = softplus(raw + dt_bias) per (token, head), 32-bit; returns
+    (decay [T, H * n_state] = exp(-rate[h] * dt) for every key channel, v [T, H * dv] = dt * x). raw [T, >= H] and x
+    [T, >= H * dv] are 32-bit rows, possibly column ranges of wider matrices."""
+    T = raw.shape[0]
+    ld_raw, ld_x = _rows32(raw, "raw", T, H), _rows32(x, "x", T, H * dv)
+    _need(dt_bias, "dt_bias", None, (H,)); _need(rate, "rate", torch.float32, (H,))
+    decay = torch.empty((T, H * n_state), dtype=torch.float32, device=raw.device)
+    v = torch.empty((T, H * dv), dtype=torch.float32, device=raw.device)
+    _call(_lib().bl_ssd_prep, _p(raw), ld_raw, _p(dt_bias), _dt(dt_bias), _p(rate), _p(x), ld_x, _p(decay), _p(v), T, H, n_state, dv, _stream())
+    return decay, v
+
+
+def gated_group_norm(o: torch.Tensor, x: Optional[torch.Tensor], skip: Optional[torch.Tensor], dv: int, z: Optional[torch.Tensor],
+                     weight: Optional[torch.Tensor], n_parts: int, eps: float, out: torch.Tensor) -> None:
+    """out = rms_norm_in_parts((o + skip[c // dv] * x) * silu(z)) * weight: the gate stands IN FRONT of the norm, and each of
+    `n_parts` equal parts of a row is normed by its own root mean square. o [T, width] 32-bit; x, z: 32-bit rows (column
+    ranges allowed); x with skip, z and weight may each be None."""
+    T, width = o.shape
+    _need(o, "o", torch.float32); _need(out, "out", None, (T, width))
+    ld_x = _rows32(x, "x", T, width) if x is not None else 0
+    ld_z = _rows32(z, "z", T, width) if z is not None else 0
+    if x is not None:
+        _need(skip, "skip", None, (width // dv,))
+    if weight is not None:
+        _need(weight, "weight", None, (width,))
+    _call(_lib().bl_gated_group_norm, _p(o), _p(x), ld_x, _p(skip), _vec_dt(skip), dv, _p(z), ld_z, _p(weight), _vec_dt(weight),
+          _p(out), _dt(out), T, width, n_parts, ctypes.c_float(eps), _stream())
+
+
+def add_scaled_pair(x: torch.Tensor, a: torch.Tensor, ca: float, b: torch.Tensor, cb: float) -> None:
+    """x += ca * a + cb * b (32-bit): two sublayer results that join the stream with a constant factor each."""
+    _need(x, "x", torch.float32); _need(a, "a", torch.float32, tuple(x.shape)); _need(b, "b", torch.float32, tuple(x.shape))
+    _call(_lib().bl_add_scaled_pair, _p(x), _p(a), ctypes.c_float(ca), _p(b), ctypes.c_float(cb), ctypes.c_longlong(x.numel()), _stream())
+
+
+def add_row_gated(x: torch.Tensor, a: torch.Tensor, gate: torch.Tensor) -> None:
+    """x[r] += sigmoid(gate[r, 0]) * a[r] (32-bit; gate: rows of a 32-bit matrix, its first column the logit)."""
+    rows, d = x.shape
+    _need(x, "x", torch.float32); _need(a, "a", torch.float32, (rows, d))
+    ld = _rows32(gate, "gate", rows, 1)
+    _call(_lib().bl_add_row_gated, _p(x), _p(a), _p(gate), ctypes.c_longlong(ld), rows, d, _stream())
+
+
+def xielu_args(p: float, q: float, device) -> torch.Tensor:
+    """The two numbers the xIELU kernel reads, from the learned p and q: {softplus(p), 1/2 + softplus(q)}, 32-bit."""
+    sp = lambda v: float(torch.nn.functional.softplus(torch.tensor(v, dtype=torch.float64)))
+    return torch.tensor([sp(p), 0.5 + sp(q)], dtype=torch.float32, device=device)
+
+
+def xielu(x: torch.Tensor, out: torch.Tensor, args: torch.Tensor) -> None:
+    """out = xIELU(x) on 32-bit sums (rows contiguous; column ranges allowed): v > 0: args[0] v^2 + v / 2, else
+    args[1] (e^v - 1 - v) + v / 2."""
+    rows, cols = out.shape
+    ld = _rows32(x, "x", rows, cols)
+    _need(args, "args", torch.float32, (2,))
+    if out.stride(1) != 1:
+        raise KernelError("xielu: out must have contiguous rows")
+    _call(_lib().bl_xielu, _p(x), ctypes.c_longlong(ld), _p(out), _dt(out), ctypes.c_longlong(out.stride(0)), rows, cols, _p(args), _stream())
