@@ -7,9 +7,10 @@ from .kavotar_config import KavotarConfig
 from .miforax_config import MiforaxConfig
 from .dapuzen_config import DapuzenConfig
 from .gipinex_config import GipinexConfig
+from .zuvevik_config import ZuvevikConfig
 
 __all__ = [
-    "ConfigError", "Qwen2Config", "FezopelConfig", "KavotarConfig", "MiforaxConfig", "DapuzenConfig", "GipinexConfig", "architecture_name", "read_config_json", "Architecture",
+    "ConfigError", "Qwen2Config", "FezopelConfig", "KavotarConfig", "MiforaxConfig", "DapuzenConfig", "GipinexConfig", "ZuvevikConfig", "architecture_name", "read_config_json", "Architecture",
     "register_architecture", "unregister_architecture", "registered_architectures",
     "resolve_architecture", "load_config", "EngineOptions",
 ]

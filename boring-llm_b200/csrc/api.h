@@ -200,25 +200,27 @@ int bl_attention_decode_tail(const void* q, const void* k_cache, const void* v_c
                              int n_splits, float* scratch, int* counters, void* out, int H, int KV, int dh, int page_size,
                              int window, float scale, const void* sinks, int sink_dtype, const float* gate, int ld_gate,
                              void* stream);
-// The tcgen05 prompt kernel, the TMA-fed decode kernel and the `mma.sync` kernels with a cap c > 0 on the scaled scores as well, s <- c tanh(s / c), before the softmax (0: none).
+// The tcgen05 prompt kernel, the TMA-fed decode kernel and the `mma.sync` kernels with a cap c > 0 on the scaled scores as well, s <- c tanh(s / c),
+// before the softmax (0: none). gate_dim n > 0: the gate holds a logit per channel, head h's n = dh logits at columns h * n .. of a token's row
+// (rows of a multiple of 4 floats, 16-byte aligned; the plain kernel: any); 0: one logit per head.
 int bl_attention_prefill_cap(const void* q, const void* k_cache, const void* v_cache, const int* cu_q,
                              const int* ctx_len, const int* block_table, int max_pages, const int* tiles, int n_tiles,
                              void* out, int H, int KV, int dh, int page_size, int window, float scale,
-                             const void* sinks, int sink_dtype, const float* gate, int ld_gate, float softcap, void* stream);
+                             const void* sinks, int sink_dtype, const float* gate, int ld_gate, int gate_dim, float softcap, void* stream);
 int bl_attention_prefill_tc_cap(const void* q, const void* k_cache, const void* v_cache, const int* cu_q,
                                 const int* ctx_len, const int* block_table, int max_pages, const int* tiles, int n_tiles,
                                 void* out, int T, int n_pages, int H, int KV, int dh, int page_size, int window, float scale,
-                                const void* sinks, int sink_dtype, const float* gate, int ld_gate, float softcap, void* stream);
+                                const void* sinks, int sink_dtype, const float* gate, int ld_gate, int gate_dim, float softcap, void* stream);
 int bl_attention_decode_tma_cap(const void* q, const void* k_cache, const void* v_cache, int n_pages, const int* cu_q,
                                 const int* ctx_len, const int* block_table, int max_pages, const int* reqs, int n,
                                 int n_splits, void* out, int H, int KV, int dh, int page_size, int window, float scale,
-                                int early, const void* sinks, int sink_dtype, const float* gate, int ld_gate, float softcap,
+                                int early, const void* sinks, int sink_dtype, const float* gate, int ld_gate, int gate_dim, float softcap,
                                 void* stream);
 int bl_attention_decode_cap(const void* q, const void* k_cache, const void* v_cache, const int* cu_q,
                             const int* ctx_len, const int* block_table, int max_pages, const int* reqs, int n,
                             int n_splits, float* scratch, int* counters, void* out, int H, int KV, int dh, int page_size,
                             int window, float scale, const void* sinks, int sink_dtype, const float* gate, int ld_gate,
-                            float softcap, void* stream);
+                            int gate_dim, float softcap, void* stream);
 int bl_attention_decode_tma_tail(const void* q, const void* k_cache, const void* v_cache, int n_pages, const int* cu_q,
                                  const int* ctx_len, const int* block_table, int max_pages, const int* reqs, int n,
                                  int n_splits, void* out, int H, int KV, int dh, int page_size, int window, float scale,
@@ -239,7 +241,7 @@ int bl_attention_plain_ext(const void* q, const void* k_cache, const void* v_cac
 int bl_attention_plain_cap(const void* q, const void* k_cache, const void* v_cache, int dtype,
                            const int* tok_req, const int* cu_q, const int* ctx_len, const int* block_table,
                            int max_pages, void* out, int T, int H, int KV, int dh, int dv, int page_size, int window,
-                           float scale, const void* sinks, int sink_dtype, const float* gate, int ld_gate, float softcap, void* stream);
+                           float scale, const void* sinks, int sink_dtype, const float* gate, int ld_gate, int gate_dim, float softcap, void* stream);
 
 // y[r, :] = (x[src, :] - mean) / sqrt(var + eps) * w + b (b may be null), src = row_idx ? row_idx[r] : r; var is the
 // mean of the squared deviations; statistics in 32-bit.
@@ -367,6 +369,18 @@ int bl_qk_norm_rope_write_scope(const float* proj, int ld, int off_k, int off_v,
                                 const int* tok_req, const int* block_table, int max_pages, const float* inv_freq,
                                 int rot_half, int pair_layout, void* q_out, void* k_cache, void* v_cache, int dtype, int T,
                                 int H, int KV, int dk, int dv, int page_size, const float* q_head_scale, void* stream);
+// ... with heads that are padded with zeros, and values blended with those of another layer (qk_norm_rope.cu). norm_q,
+// norm_k > 0: how many values the whole-row norms average over (0: all of H * dk, KV * dk). v_first (null: none), 32-bit rows
+// ld_first apart: values of the same tokens, heads of first_dv values first_places apart; the cached values become
+// (1 - lambda) v + lambda v_first, matched channel by channel over the flat row (this layer's heads have dv_real values, then
+// zeros up to dv); lambda: one number on the device.
+int bl_qk_norm_rope_write_ext(const float* proj, int ld, int off_k, int off_v, const void* q_norm_w, int qw_dtype,
+                              const void* k_norm_w, int kw_dtype, float eps, int per_head, const int* positions,
+                              const int* tok_req, const int* block_table, int max_pages, const float* inv_freq,
+                              int rot_half, int pair_layout, void* q_out, void* k_cache, void* v_cache, int dtype, int T,
+                              int H, int KV, int dk, int dv, int page_size, const float* q_head_scale, int norm_q, int norm_k,
+                              const float* v_first, int ld_first, int first_dv, int first_places, int dv_real, const void* lambda,
+                              int lambda_dtype, void* stream);
 // out[m, n] = exp(-exp(u[m, :] . W[n, :] + bias[n])), u = tanh(x) where x_tanh != 0 (x: 32-bit rows ldx apart).
 int bl_gemm_plain_decay_exp(const float* x, int ldx, int x_tanh, const void* w, int w_dtype, const void* bias, int bias_dtype,
                             float* out, int M, int N, int K, void* stream);
@@ -444,6 +458,11 @@ int bl_moe_combine_rows_some(const float* y, const int* pos, const float* wts, f
 // expert's matrix (gemm_tcgen05.cu), and bl_moe_combine_rows adds up a token's rows y[pos[t * top + k]].
 int bl_moe_plan(const int* ids, int P, int E, int tile, int max_tiles, int* pos, int* row_src, int* tile_expert, void* stream);
 int bl_gather_rows(const void* x, const int* row_src, int div, void* dst, int rows, int cols, void* stream);
+// A weight per pair on what the pair's expert READS (instead of on its result): the gathered row of pair p times wts[p]
+// (null: 1), or, for the plain products, dst [T * top, d] = x[p / top, :] * wts[p]. bl_moe_combine and its variants add the
+// results up unweighted when their wts is null.
+int bl_gather_rows_weighted(const void* x, const int* row_src, int div, const float* wts, void* dst, int rows, int cols, void* stream);
+int bl_scale_pairs(const void* x, int dtype, const float* wts, int T, int top, int d, void* dst, void* stream);
 int bl_gemm_tc_grouped(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K, int epilogue, int n_experts,
                        const int* tile_expert, const float* act, void* stream);
 int bl_moe_combine_rows(const float* y, const int* pos, const float* wts, float* out, int T, int top, int d, int add, void* stream);
@@ -518,6 +537,20 @@ int bl_attention_mixed_prefill(const void* q, const void* k_cache, const float* 
 int bl_attention_mixed_decode(const void* q, const void* k_cache, const float* k_rms, const int* cu_q, const int* ctx_len,
                               const int* block_table, int max_pages, const int* reqs, int n, int n_splits, void* out, int H, int KV, int dh,
                               int page_size, float scale, const float* slopes, const float* gate, int ld_gate, void* stream);
+
+// A residual of n streams, x [n][rows][d] 32-bit, x_stride floats apart (0: all of them are the same rows), hyper.cu. With
+// `write` (b [n], then M [n, n] indexed [from, to], 32-bit): x'_t = sum_s M[s, t] x_s + b[t] y into x_out (null: not stored; x
+// itself: in place), where y is row t of y (y_pos null, top 1) or the sum over k < top of y_wts[t * top + k] (null: 1) times
+// row y_pos[t * top + k] (null: row t * top + k; negative: nothing). With h: the row sum_s read[s] x'_s (read null: the plain
+// sum), divided by its root mean square and times w (w null: as it is), of tokens row_idx[r] (null: r), r < rows.
+int bl_hyper_step(const float* x, long long x_stride, float* x_out, long long out_stride, int n, const float* write, const float* y,
+                  const int* y_pos, const float* y_wts, int top, const float* read, const void* w, int w_dtype, float eps, void* h,
+                  int h_dtype, const int* row_idx, int rows, int d, void* stream);
+// out[t, :] = table[token, :] + pairs[row, :], row = (previous token * mul_prev + token * mul_cur) mod buckets (the sequence's
+// first token: row `buckets`). prev_tokens [slots] holds each request's last token between steps; it is read and written here.
+int bl_embed_pairs(const void* table, const void* pairs, int dtype, const int* ids, const int* positions, const int* tok_req,
+                   const int* cu_q, const int* slots, int* prev_tokens, long long mul_prev, long long mul_cur, long long buckets,
+                   float* out, int T, int d, void* stream);
 
 #ifdef __cplusplus
 }

@@ -426,8 +426,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             }
             if (n_splits == 1) {
                 const float inv = bl_attn_tail(p.tail, M, L, (size_t)q_begin, head0 + row);
+                const float4 cg = bl_gate4(p.tail, (size_t)q_begin, head0 + row, d);
                 *reinterpret_cast<uint2*>(p.out + ((size_t)q_begin * p.H + head0 + row) * DH + d) =
-                    make_uint2(pack_bf16(O.x * inv, O.y * inv), pack_bf16(O.z * inv, O.w * inv));
+                    make_uint2(pack_bf16(O.x * inv * cg.x, O.y * inv * cg.y), pack_bf16(O.z * inv * cg.z, O.w * inv * cg.w));
             } else {
                 const uint32_t owner = (uint32_t)(row % n_splits);
                 const uint32_t slot = recv + (uint32_t)((row / n_splits) * n_splits + split) * (ROWF * 4);
@@ -456,8 +457,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 O.x += a.x * f; O.y += a.y * f; O.z += a.z * f; O.w += a.w * f;
             }
             const float inv = bl_attn_tail(p.tail, M, L, (size_t)q_begin, head0 + row);
+            const float4 cg = bl_gate4(p.tail, (size_t)q_begin, head0 + row, d);
             *reinterpret_cast<uint2*>(p.out + ((size_t)q_begin * p.H + head0 + row) * DH + d) =
-                make_uint2(pack_bf16(O.x * inv, O.y * inv), pack_bf16(O.z * inv, O.w * inv));
+                make_uint2(pack_bf16(O.x * inv * cg.x, O.y * inv * cg.y), pack_bf16(O.z * inv * cg.z, O.w * inv * cg.w));
         }
     }
     cluster_sync_all();                                           // nobody leaves while a store to its shared memory may be in flight
@@ -563,7 +565,7 @@ extern "C" int bl_attention_decode_tma_tail(const void* q, const void* k_cache, 
                                             float scale, int early, const void* sinks, int sink_dtype, const float* gate,
                                             int ld_gate, void* stream) {
     return bl_attention_decode_tma_cap(q, k_cache, v_cache, n_pages, cu_q, ctx_len, block_table, max_pages, reqs, n, n_splits, out, H, KV,
-                                       dh, page_size, window, scale, early, sinks, sink_dtype, gate, ld_gate, 0.f, stream);
+                                       dh, page_size, window, scale, early, sinks, sink_dtype, gate, ld_gate, 0, 0.f, stream);
 }
 
 // ... and a cap c > 0 on the scaled scores, s <- c tanh(s / c), before the softmax (0: none).
@@ -571,7 +573,7 @@ extern "C" int bl_attention_decode_tma_cap(const void* q, const void* k_cache, c
                                            const int* ctx_len, const int* block_table, int max_pages, const int* reqs, int n,
                                            int n_splits, void* out, int H, int KV, int dh, int page_size, int window,
                                            float scale, int early, const void* sinks, int sink_dtype, const float* gate,
-                                           int ld_gate, float softcap, void* stream) {
+                                           int ld_gate, int gate_dim, float softcap, void* stream) {
     if (n <= 0) return 0;
     if (!(softcap >= 0.f)) BL_FAIL("%s: a cap on the scores must not be negative, got %g", WHO, (double)softcap);
     if (!(scale > 0.f)) BL_FAIL("%s: the scale of the scores must be positive (got %g)", WHO, (double)scale);
@@ -584,7 +586,8 @@ extern "C" int bl_attention_decode_tma_cap(const void* q, const void* k_cache, c
     p.q = (const __nv_bfloat16*)q; p.out = (__nv_bfloat16*)out; p.cu_q = cu_q; p.ctx_len = ctx_len;
     p.block_table = block_table; p.max_pages = max_pages; p.reqs = reqs; p.n_splits = n_splits;
     p.H = H; p.KV = KV; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
-    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate};
+    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate, gate_dim};
+    if (!bl_channel_gate_ok(gate, ld_gate, gate_dim, H, dh)) BL_FAIL("%s: a gate of %d channels a head in rows of %d does not fit %d heads of %d in 16-byte pieces", WHO, gate_dim, ld_gate, H, dh);
     p.cap_log2 = softcap * 1.4426950408889634f;
     CUtensorMap mk, mv;
     if (bl_make_map_bf16(WHO, &mk, k_cache, (long long)n_pages * KV * PAGE, dh, PAGE, 64)) return 1;

@@ -467,8 +467,10 @@ attention_mma_kernel(const AttnParams p) {
             const float inv = bl_attn_tail(p.tail, m[h], l[h], (size_t)(q_begin + tok[h]), head[h]);
             __nv_bfloat16* op = out_row(p, (size_t)(q_begin + tok[h]), head[h], vh, DH) + 2 * t;
 #pragma unroll
-            for (int n = 0; n < DH / 8; ++n)
-                *reinterpret_cast<unsigned*>(op + n * 8) = pack_bf16(o[n][2 * h] * inv, o[n][2 * h + 1] * inv);
+            for (int n = 0; n < DH / 8; ++n) {
+                const float2 cg = bl_gate2(p.tail, (size_t)(q_begin + tok[h]), head[h], n * 8 + 2 * t);
+                *reinterpret_cast<unsigned*>(op + n * 8) = pack_bf16(o[n][2 * h] * inv * cg.x, o[n][2 * h + 1] * inv * cg.y);
+            }
         }
         return;
     }
@@ -520,8 +522,9 @@ attention_mma_kernel(const AttnParams p) {
             const int hd = head0 + row;
             if (p.n_splits == 1) {
                 const float inv = bl_attn_tail(p.tail, M, L, (size_t)q_tok, hd);
+                const float4 cg = bl_gate4(p.tail, (size_t)q_tok, hd, d);
                 *reinterpret_cast<uint2*>(out_row(p, (size_t)q_tok, hd, vh, DH) + d) =
-                    make_uint2(pack_bf16(O.x * inv, O.y * inv), pack_bf16(O.z * inv, O.w * inv));
+                    make_uint2(pack_bf16(O.x * inv * cg.x, O.y * inv * cg.y), pack_bf16(O.z * inv * cg.z, O.w * inv * cg.w));
             } else if (p.part_o == nullptr) {                             // the slices are the blocks of one cluster: the partial result stays here
                 *reinterpret_cast<float4*>(cp_o + row * DH + d) = O;
                 if (d == 0) *reinterpret_cast<float2*>(cp_ml + row * 2) = make_float2(M, L);
@@ -563,8 +566,9 @@ attention_mma_kernel(const AttnParams p) {
                 O.x += po[s2].x * f; O.y += po[s2].y * f; O.z += po[s2].z * f; O.w += po[s2].w * f;
             }
             const float inv = bl_attn_tail(p.tail, M, L, (size_t)q_tok, head0 + row);
+            const float4 cg = bl_gate4(p.tail, (size_t)q_tok, head0 + row, d);
             *reinterpret_cast<uint2*>(out_row(p, (size_t)q_tok, head0 + row, vh, DH) + d) =
-                make_uint2(pack_bf16(O.x * inv, O.y * inv), pack_bf16(O.z * inv, O.w * inv));
+                make_uint2(pack_bf16(O.x * inv * cg.x, O.y * inv * cg.y), pack_bf16(O.z * inv * cg.z, O.w * inv * cg.w));
         }
         cluster_sync_all();                                           // no block leaves while another may still read its partial result
         return;
@@ -651,8 +655,9 @@ attention_mma_kernel(const AttnParams p) {
             }
         }
         const float inv = bl_attn_tail(p.tail, sM[row], sL[row], (size_t)q_tok, head0 + row);
+        const float4 cg = bl_gate4(p.tail, (size_t)q_tok, head0 + row, d);
         __nv_bfloat16* dst = out_row(p, (size_t)q_tok, head0 + row, vh, DH) + d;
-        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(O.x * inv, O.y * inv), pack_bf16(O.z * inv, O.w * inv));
+        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(O.x * inv * cg.x, O.y * inv * cg.y), pack_bf16(O.z * inv * cg.z, O.w * inv * cg.w));
     }
 }
 
@@ -765,7 +770,7 @@ extern "C" int bl_attention_prefill_tail(const void* q, const void* k_cache, con
                                          float scale, const void* sinks, int sink_dtype, const float* gate, int ld_gate,
                                          void* stream) {
     return bl_attention_prefill_cap(q, k_cache, v_cache, cu_q, ctx_len, block_table, max_pages, tiles, n_tiles, out, H, KV, dh,
-                                    page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0.f, stream);
+                                    page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0, 0.f, stream);
 }
 
 // ... and a cap c > 0 on the scaled scores, s <- c tanh(s / c), before the softmax (0: none).
@@ -773,7 +778,7 @@ extern "C" int bl_attention_prefill_cap(const void* q, const void* k_cache, cons
                                         const int* ctx_len, const int* block_table, int max_pages, const int* tiles,
                                         int n_tiles, void* out, int H, int KV, int dh, int page_size, int window,
                                         float scale, const void* sinks, int sink_dtype, const float* gate, int ld_gate,
-                                        float softcap, void* stream) {
+                                        int gate_dim, float softcap, void* stream) {
     if (n_tiles <= 0) return 0;
     if (!(softcap >= 0.f)) BL_FAIL("bl_attention_prefill: a cap on the scores must not be negative, got %g", (double)softcap);
     if (check(H, KV, dh, page_size, max_pages, window, scale)) return 1;
@@ -783,7 +788,8 @@ extern "C" int bl_attention_prefill_cap(const void* q, const void* k_cache, cons
     p.work = tiles; p.part_o = nullptr; p.part_ml = nullptr; p.counters = nullptr; p.n_splits = 1; p.H = H; p.KV = KV; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.cap_log2 = softcap * 1.4426950408889634f;
-    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate};
+    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate, gate_dim};
+    if (!bl_channel_gate_ok(gate, ld_gate, gate_dim, H, dh)) BL_FAIL("%s: a gate of %d channels a head in rows of %d does not fit %d heads of %d in 16-byte pieces", "bl_attention_prefill", gate_dim, ld_gate, H, dh);
     if ((long long)n_tiles * H > 2147483647LL) BL_FAIL("bl_attention_prefill: %d tiles x %d heads are more blocks than a launch takes", n_tiles, H);
     return dispatch<false>(dh, p, dim3(n_tiles * H, 1, 1), (cudaStream_t)stream);
 }
@@ -808,14 +814,14 @@ extern "C" int bl_attention_decode_tail(const void* q, const void* k_cache, cons
                                         int page_size, int window, float scale, const void* sinks, int sink_dtype,
                                         const float* gate, int ld_gate, void* stream) {
     return bl_attention_decode_cap(q, k_cache, v_cache, cu_q, ctx_len, block_table, max_pages, reqs, n, n_splits, scratch, counters,
-                                   out, H, KV, dh, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0.f, stream);
+                                   out, H, KV, dh, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0, 0.f, stream);
 }
 
 extern "C" int bl_attention_decode_cap(const void* q, const void* k_cache, const void* v_cache, const int* cu_q,
                                        const int* ctx_len, const int* block_table, int max_pages, const int* reqs, int n,
                                        int n_splits, float* scratch, int* counters, void* out, int H, int KV, int dh,
                                        int page_size, int window, float scale, const void* sinks, int sink_dtype,
-                                       const float* gate, int ld_gate, float softcap, void* stream) {
+                                       const float* gate, int ld_gate, int gate_dim, float softcap, void* stream) {
     if (n <= 0) return 0;
     if (!(softcap >= 0.f)) BL_FAIL("bl_attention_decode: a cap on the scores must not be negative, got %g", (double)softcap);
     if (check(H, KV, dh, page_size, max_pages, window, scale)) return 1;
@@ -832,7 +838,8 @@ extern "C" int bl_attention_decode_cap(const void* q, const void* k_cache, const
     p.counters = counters;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.cap_log2 = softcap * 1.4426950408889634f;
-    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate};
+    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate, gate_dim};
+    if (!bl_channel_gate_ok(gate, ld_gate, gate_dim, H, dh)) BL_FAIL("%s: a gate of %d channels a head in rows of %d does not fit %d heads of %d in 16-byte pieces", "bl_attention_decode", gate_dim, ld_gate, H, dh);
     const int G = H / KV;
     return dispatch<true>(dh, p, dim3(n_splits, KV * ((G + 15) / 16), n), (cudaStream_t)stream);
 }
@@ -854,7 +861,7 @@ extern "C" int bl_attention_prefill_talk(const void* q, const void* k_cache, con
     p.out = (__nv_bfloat16*)spread; p.cu_q = cu_q; p.ctx_len = ctx_len; p.block_table = block_table; p.max_pages = max_pages;
     p.work = tiles; p.n_splits = 1; p.H = H; p.KV = KV; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f;
-    p.tail = BlAttnTail{nullptr, 0, nullptr, 0};
+    p.tail = BlAttnTail{nullptr, 0, nullptr, 0, 0};
     p.chunk = chunk; p.head_scale = head_scale; p.spread = 1;
     if ((long long)n_tiles * H > 2147483647LL) BL_FAIL("bl_attention_prefill_talk: %d tiles x %d heads are more blocks than a launch takes", n_tiles, H);
     return dispatch<false>(dh, p, dim3(n_tiles * H, KV, 1), (cudaStream_t)stream);      // y: the value head's shift
@@ -873,7 +880,7 @@ extern "C" int bl_attention_decode_talk(const void* q, const void* k_cache, cons
     p.out = (__nv_bfloat16*)spread; p.cu_q = cu_q; p.ctx_len = ctx_len; p.block_table = block_table; p.max_pages = max_pages;
     p.work = reqs; p.n_splits = n_splits; p.H = H; p.KV = KV; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f;
-    p.tail = BlAttnTail{nullptr, 0, nullptr, 0};
+    p.tail = BlAttnTail{nullptr, 0, nullptr, 0, 0};
     p.chunk = chunk; p.head_scale = head_scale; p.spread = 1;
     const int G = H / KV;
     if ((long long)KV * KV * ((G + 15) / 16) > 65535) BL_FAIL("bl_attention_decode_talk: %d key/value heads are too many for one launch", KV);

@@ -7,7 +7,7 @@
 // at its first visible key. This is the 32-bit path's attention and the twin of the fast kernels.
 // Options (bl_attention_plain_ext): values of another head size than the keys; a sink per head, a learned score that
 // joins the softmax's denominator once, unscaled, without a value; a gate per (token, head) whose sigmoid multiplies
-// the head's output; a cap c on the scores, s <- c tanh(s / c), applied to the scaled score before the softmax.
+// the head's output, or one per (token, head, channel); a cap c on the scores, s <- c tanh(s / c), applied to the scaled score before the softmax.
 #include "common.cuh"
 #include "api.h"
 
@@ -22,7 +22,7 @@ attention_plain_kernel(const TT* __restrict__ q, const TT* __restrict__ kc, cons
                        const int* __restrict__ tok_req, const int* __restrict__ cu_q,
                        const int* __restrict__ ctx_len, const int* __restrict__ block_table, int max_pages,
                        TT* __restrict__ out, int T, int H, int KV, int dh, int dv, int page_size, int window,
-                       float scale, const void* __restrict__ sinks, int sink_dtype, const float* gate, int ld_gate, float softcap) {
+                       float scale, const void* __restrict__ sinks, int sink_dtype, const float* gate, int ld_gate, int gate_dim, float softcap) {
     __shared__ float qs[WARPS][MAX_DH];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int item = blockIdx.x * WARPS + warp;
@@ -85,11 +85,12 @@ attention_plain_kernel(const TT* __restrict__ q, const TT* __restrict__ kc, cons
     }
     TT* orow = out + ((size_t)t * H + h) * dv;
     float inv = l > 0.f ? 1.0f / l : 0.f;
-    if (gate) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ld_gate + h]));
+    if (gate && gate_dim == 0) inv *= bl_sigmoid(gate[(size_t)t * ld_gate + h]);
+    const float* crow = gate && gate_dim ? gate + (size_t)t * ld_gate + (size_t)h * gate_dim : nullptr;
 #pragma unroll
     for (int i = 0; i < MAX_DH / 32; ++i) {
         const int d = lane + 32 * i;
-        if (d < dv) bl_store(orow + d, acc[i] * inv);
+        if (d < dv) bl_store(orow + d, crow ? acc[i] * inv * bl_sigmoid(crow[d]) : acc[i] * inv);
     }
 }
 
@@ -109,17 +110,18 @@ extern "C" int bl_attention_plain_ext(const void* q, const void* k_cache, const 
                                       int dh, int dv, int page_size, int window, float scale, const void* sinks,
                                       int sink_dtype, const float* gate, int ld_gate, void* stream) {
     return bl_attention_plain_cap(q, k_cache, v_cache, dtype, tok_req, cu_q, ctx_len, block_table, max_pages, out, T, H, KV,
-                                  dh, dv, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0.f, stream);
+                                  dh, dv, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0, 0.f, stream);
 }
 
 extern "C" int bl_attention_plain_cap(const void* q, const void* k_cache, const void* v_cache, int dtype,
                                       const int* tok_req, const int* cu_q, const int* ctx_len,
                                       const int* block_table, int max_pages, void* out, int T, int H, int KV,
                                       int dh, int dv, int page_size, int window, float scale, const void* sinks,
-                                      int sink_dtype, const float* gate, int ld_gate, float softcap, void* stream) {
+                                      int sink_dtype, const float* gate, int ld_gate, int gate_dim, float softcap, void* stream) {
     if (T <= 0) return 0;
     if (!(softcap >= 0.f)) BL_FAIL("bl_attention_plain: a cap on the scores must not be negative, got %g", (double)softcap);
     if (dv <= 0 || dv > MAX_DH) BL_FAIL("bl_attention_plain: value head size %d is outside 1..%d", dv, MAX_DH);
+    if (gate_dim && (!gate || gate_dim != dv || ld_gate < H * dv)) BL_FAIL("bl_attention_plain: a gate of %d channels a head in rows of %d for %d heads of %d", gate_dim, ld_gate, H, dv);
     if (gate && ld_gate < H) BL_FAIL("bl_attention_plain: gate rows of %d hold fewer than %d heads", ld_gate, H);
     if (H <= 0 || KV <= 0 || H % KV != 0) BL_FAIL("bl_attention_plain: %d heads cannot share %d key/value heads", H, KV);
     if (dh <= 0 || dh > MAX_DH) BL_FAIL("bl_attention_plain: head size %d is outside 1..%d", dh, MAX_DH);
@@ -129,11 +131,11 @@ extern "C" int bl_attention_plain_cap(const void* q, const void* k_cache, const 
     if (dtype == BL_F32)
         attention_plain_kernel<float><<<blocks, WARPS * 32, 0, s>>>((const float*)q, (const float*)k_cache,
             (const float*)v_cache, tok_req, cu_q, ctx_len, block_table, max_pages, (float*)out, T, H, KV, dh, dv,
-            page_size, window, scale, sinks, sink_dtype, gate, ld_gate, softcap);
+            page_size, window, scale, sinks, sink_dtype, gate, ld_gate, gate_dim, softcap);
     else if (dtype == BL_BF16)
         attention_plain_kernel<__nv_bfloat16><<<blocks, WARPS * 32, 0, s>>>((const __nv_bfloat16*)q,
             (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, tok_req, cu_q, ctx_len, block_table,
-            max_pages, (__nv_bfloat16*)out, T, H, KV, dh, dv, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, softcap);
+            max_pages, (__nv_bfloat16*)out, T, H, KV, dh, dv, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, gate_dim, softcap);
     else
         BL_FAIL("bl_attention_plain: unknown dtype %d", dtype);
     BL_CHECK_LAUNCH("bl_attention_plain");

@@ -571,6 +571,18 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             if (ok && valid) {
                 const float inv = bl_attn_tail(p.tail, m, l, (size_t)(q_begin + tok0 + row), head);
                 __nv_bfloat16* dst = p.out + ((size_t)(q_begin + tok0 + row) * p.H + head) * DH;
+                // (the row's channel gate, if there is one, in a loop of its own: 16 channels at a time keep the registers as they were)
+                if (p.tail.gate_dim) {
+#pragma unroll
+                    for (int c = 0; c < DH; c += 16) {
+                        asm volatile("" ::: "memory");
+#pragma unroll
+                        for (int j = c; j < c + 16; j += 4) {
+                            const float4 cg = bl_gate4(p.tail, (size_t)(q_begin + tok0 + row), head, j);
+                            o[j] *= cg.x; o[j + 1] *= cg.y; o[j + 2] *= cg.z; o[j + 3] *= cg.w;
+                        }
+                    }
+                }
 #pragma unroll
                 for (int j = 0; j < DH; j += 8)
                     *reinterpret_cast<uint4*>(dst + j) = make_uint4(pack_bf16(o[j] * inv, o[j + 1] * inv), pack_bf16(o[j + 2] * inv, o[j + 3] * inv),
@@ -598,6 +610,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 float r[DH / 2];
 #pragma unroll
                 for (int j = 0; j < DH / 2; ++j) r[j] = (grp ? o[DH / 2 + j] : o[j]) * wa + theirs[row * MERGE_ROW + j] * wo;
+                if (p.tail.gate_dim) {
+#pragma unroll
+                    for (int j = 0; j < DH / 2; j += 4) {
+                        const float4 cg = bl_gate4(p.tail, (size_t)(q_begin + tok0 + row), head, grp * (DH / 2) + j);
+                        r[j] *= cg.x; r[j + 1] *= cg.y; r[j + 2] *= cg.z; r[j + 3] *= cg.w;
+                    }
+                }
                 __nv_bfloat16* dst = p.out + ((size_t)(q_begin + tok0 + row) * p.H + head) * DH + grp * (DH / 2);
 #pragma unroll
                 for (int j = 0; j < DH / 2; j += 8)
@@ -657,7 +676,7 @@ extern "C" int bl_attention_prefill_tc_tail(const void* q, const void* k_cache, 
                                             int window, float scale, const void* sinks, int sink_dtype, const float* gate,
                                             int ld_gate, void* stream) {
     return bl_attention_prefill_tc_cap(q, k_cache, v_cache, cu_q, ctx_len, block_table, max_pages, tiles, n_tiles, out, T, n_pages, H, KV,
-                                       dh, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0.f, stream);
+                                       dh, page_size, window, scale, sinks, sink_dtype, gate, ld_gate, 0, 0.f, stream);
 }
 
 // ... and a cap c > 0 on the scaled scores, s <- c tanh(s / c), before the softmax (0: none; the kernel without it).
@@ -665,7 +684,7 @@ extern "C" int bl_attention_prefill_tc_cap(const void* q, const void* k_cache, c
                                            const int* ctx_len, const int* block_table, int max_pages, const int* tiles,
                                            int n_tiles, void* out, int T, int n_pages, int H, int KV, int dh, int page_size,
                                            int window, float scale, const void* sinks, int sink_dtype, const float* gate,
-                                           int ld_gate, float softcap, void* stream) {
+                                           int ld_gate, int gate_dim, float softcap, void* stream) {
     if (n_tiles <= 0) return 0;
     if (!(softcap >= 0.f)) BL_FAIL("bl_attention_prefill_tc: a cap on the scores must not be negative, got %g", (double)softcap);
     if ((dh != 64 && dh != 128) || page_size != PAGE)
@@ -679,7 +698,8 @@ extern "C" int bl_attention_prefill_tc_cap(const void* q, const void* k_cache, c
     Params p;
     p.out = (__nv_bfloat16*)out; p.cu_q = cu_q; p.ctx_len = ctx_len; p.block_table = block_table; p.max_pages = max_pages;
     p.tiles = tiles; p.H = H; p.KV = KV; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
-    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate};
+    p.tail = BlAttnTail{sinks, sink_dtype, gate, ld_gate, gate_dim};
+    if (!bl_channel_gate_ok(gate, ld_gate, gate_dim, H, dh)) BL_FAIL("%s: a gate of %d channels a head in rows of %d does not fit %d heads of %d in 16-byte pieces", "bl_attention_prefill_tc", gate_dim, ld_gate, H, dh);
     p.cap_log2 = softcap * 1.4426950408889634f;
     if (softcap > 0.f) {
         if (dh == 64) return launch<Shape<64, 2>, true>(q, k_cache, v_cache, p, n_tiles, T, n_pages, (cudaStream_t)stream);

@@ -111,8 +111,27 @@ __device__ __forceinline__ float bl_xielu(float v, float ap, float an) {
 // What may follow the softmax of an attention row: a sink per head (a learned score whose exponential joins the
 // denominator once, unscaled, with no value) and a gate per (token, head) whose sigmoid multiplies the row's output.
 // bl_attn_tail returns the factor for the row's unnormalised output, given the row's maximum m in the base-2 domain
-// (score * scale * log2 e) and the sum l of 2^(score - m). Null pointers: a plain 1 / l.
-struct BlAttnTail { const void* sinks; int sink_dtype; const float* gate; int ld_gate; };
+// (score * scale * log2 e) and the sum l of 2^(score - m). Null pointers: a plain 1 / l. gate_dim n > 0: the gate has a
+// logit per channel instead, head h's n logits at columns h * n .. of the token's row; it is then not part of the factor,
+// and the kernels multiply what they write by bl_gate2 / bl_gate4 (channels d, d + 1, ... of a head).
+struct BlAttnTail { const void* sinks; int sink_dtype; const float* gate; int ld_gate; int gate_dim; };
+__device__ __forceinline__ float bl_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+// The same with the hardware's exponential and division (relative error around 1e-6), for results rounded to bfloat16.
+__device__ __forceinline__ float bl_sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float2 bl_gate2(const BlAttnTail& t, size_t tok, int head, int d) {
+    if (t.gate_dim == 0) return make_float2(1.f, 1.f);
+    const float2 g = *reinterpret_cast<const float2*>(t.gate + tok * (size_t)t.ld_gate + (size_t)head * t.gate_dim + d);
+    return make_float2(bl_sigmoid_fast(g.x), bl_sigmoid_fast(g.y));
+}
+__device__ __forceinline__ float4 bl_gate4(const BlAttnTail& t, size_t tok, int head, int d) {
+    if (t.gate_dim == 0) return make_float4(1.f, 1.f, 1.f, 1.f);
+    const float4 g = *reinterpret_cast<const float4*>(t.gate + tok * (size_t)t.ld_gate + (size_t)head * t.gate_dim + d);
+    return make_float4(bl_sigmoid_fast(g.x), bl_sigmoid_fast(g.y), bl_sigmoid_fast(g.z), bl_sigmoid_fast(g.w));
+}
+// What the tensor-core kernels ask of a gate per channel: the head's size, rows that hold all heads, 16-byte pieces.
+inline bool bl_channel_gate_ok(const float* gate, int ld_gate, int gate_dim, int H, int dh) {
+    return gate_dim == 0 || (gate != nullptr && gate_dim == dh && ld_gate >= H * dh && ld_gate % 4 == 0 && ((uintptr_t)gate & 15) == 0);
+}
 __device__ __forceinline__ float bl_attn_tail(const BlAttnTail& t, float m_log2, float l, size_t tok, int head) {
     float f = 1.f;
     if (t.sinks) {
@@ -122,7 +141,7 @@ __device__ __forceinline__ float bl_attn_tail(const BlAttnTail& t, float m_log2,
         l = l * f + exp2f(sk - mm);
     }
     float inv = l > 0.f ? f / l : 0.f;
-    if (t.gate) inv *= 1.0f / (1.0f + expf(-t.gate[tok * (size_t)t.ld_gate + head]));
+    if (t.gate && t.gate_dim == 0) inv *= 1.0f / (1.0f + expf(-t.gate[tok * (size_t)t.ld_gate + head]));
     return inv;
 }
 

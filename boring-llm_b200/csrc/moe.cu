@@ -135,7 +135,18 @@ expert_gemm_plain_kernel(const TX* __restrict__ x, int x_div, const TW* __restri
     if (lane == 0) bl_store(out + (size_t)p * N + n, a);
 }
 
-// out[t, :] = (add ? out[t, :] : 0) + sum_k wts[t, k] * y[t * top + k, :], k ascending; a pair whose expert is an identity
+// dst[p, :] = x[p / top, :] * wts[p]: every pair's own row of what its expert reads.
+template <typename TT>
+__global__ void scale_pairs_kernel(const TT* __restrict__ x, const float* __restrict__ wts, int top, int d, TT* __restrict__ dst, size_t count) {
+    bl_pdl_trigger();
+    bl_pdl_wait();
+    for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < count; e += (size_t)gridDim.x * blockDim.x) {
+        const size_t p = e / d;
+        bl_store(dst + e, bl_load(x + (p / top) * d + e % d) * wts[p]);
+    }
+}
+
+// out[t, :] = (add ? out[t, :] : 0) + sum_k wts[t, k] * y[t * top + k, :] (wts null: ones), k ascending; a pair whose expert is an identity
 // expert (ids given, ids[t * top + k] >= n_real) takes x[t, :] in the place of its row of y.
 template <typename TX>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ wts, float* out, int top, int d,
@@ -147,7 +158,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
             const bool same = ids && ids[t * top + k] >= n_real;
-            acc = fmaf(wts[t * top + k], same ? bl_load(x + t * d + c) : y[(t * top + k) * d + c], acc);
+            acc = fmaf(wts ? wts[t * top + k] : 1.f, same ? bl_load(x + t * d + c) : y[(t * top + k) * d + c], acc);
         }
         out[e] = add ? out[e] + acc : acc;
     }
@@ -190,14 +201,25 @@ moe_plan_kernel(const int* __restrict__ ids, int P, int E, int tile, int max_til
 }
 
 // dst[row, :] = x[row_src[row] / div, :] (zeros where row_src is negative): the rows of a grouped product, 16 bytes a thread.
+// wts: the row is multiplied by its pair's weight wts[row_src[row]] (in 32-bit, rounded once).
 __global__ void gather_rows_kernel(const uint4* __restrict__ x, const int* __restrict__ row_src, int div, uint4* __restrict__ dst,
-                                   int rows, int vecs) {
+                                   int rows, int vecs, const float* __restrict__ wts) {
     bl_pdl_trigger();
     bl_pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < (size_t)rows * vecs; i += (size_t)gridDim.x * blockDim.x) {
         const int row = (int)(i / vecs), v = (int)(i % vecs);
         const int src = row_src[row];
-        dst[i] = src >= 0 ? x[(size_t)(src / div) * vecs + v] : make_uint4(0, 0, 0, 0);
+        uint4 val = src >= 0 ? x[(size_t)(src / div) * vecs + v] : make_uint4(0, 0, 0, 0);
+        if (wts && src >= 0) {
+            const float w = wts[src];
+            __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&val);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float2 f = __bfloat1622float2(h[j]);
+                h[j] = __floats2bfloat162_rn(f.x * w, f.y * w);
+            }
+        }
+        dst[i] = val;
     }
 }
 
@@ -213,7 +235,7 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ y, const int* 
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
             const int row = pos[t * top + k];
-            acc = fmaf(wts[t * top + k], row < 0 ? (x ? bl_load(x + t * d + c) : 0.f) : y[(size_t)row * d + c], acc);
+            acc = fmaf(wts ? wts[t * top + k] : 1.f, row < 0 ? (x ? bl_load(x + t * d + c) : 0.f) : y[(size_t)row * d + c], acc);
         }
         out[e] = add ? out[e] + acc : acc;
     }
@@ -327,13 +349,18 @@ extern "C" int bl_moe_plan(const int* ids, int P, int E, int tile, int max_tiles
 
 // dst[row, :] = x[row_src[row] / div, :], zeros where row_src[row] < 0; rows of `cols` bfloat16 values, cols a multiple of 8.
 extern "C" int bl_gather_rows(const void* x, const int* row_src, int div, void* dst, int rows, int cols, void* stream) {
+    return bl_gather_rows_weighted(x, row_src, div, nullptr, dst, rows, cols, stream);
+}
+
+// wts (null: none), one per pair: the row of pair p is multiplied by wts[p].
+extern "C" int bl_gather_rows_weighted(const void* x, const int* row_src, int div, const float* wts, void* dst, int rows, int cols, void* stream) {
     if (rows <= 0) return 0;
     if (cols <= 0 || cols % 8 != 0 || div <= 0 || (((uintptr_t)x | (uintptr_t)dst) & 15)) BL_FAIL("bl_gather_rows: rows of %d values", cols);
     const int vecs = cols / 8;
     const size_t n = (size_t)rows * vecs;
     const int blocks = (int)((n + 255) / 256 < 4096 ? (n + 255) / 256 : 4096);
     BL_CUDA(bl_launch_dependent(gather_rows_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const uint4*)x, row_src, div,
-                                (uint4*)dst, rows, vecs));
+                                (uint4*)dst, rows, vecs, wts));
     BL_CHECK_LAUNCH("bl_gather_rows");
     return 0;
 }
@@ -365,5 +392,21 @@ extern "C" int bl_table_route(const int* table, const int* tokens, int T, int to
     if (top <= 0) BL_FAIL("bl_table_route: %d experts a token", top);
     BL_CUDA(bl_launch_dependent(table_route_kernel, dim3((T * top + 127) / 128), dim3(128), 0, (cudaStream_t)stream, table, tokens, T, top, ids, wts));
     BL_CHECK_LAUNCH("bl_table_route");
+    return 0;
+}
+
+// dst [T * top, d] = x[p / top, :] * wts[p], x and dst of one dtype (the plain products' form of bl_gather_rows_weighted).
+extern "C" int bl_scale_pairs(const void* x, int dtype, const float* wts, int T, int top, int d, void* dst, void* stream) {
+    if (T <= 0) return 0;
+    if (top <= 0 || d <= 0) BL_FAIL("bl_scale_pairs: bad sizes top=%d d=%d", top, d);
+    const size_t count = (size_t)T * top * d;
+    const int blocks = (int)((count + 255) / 256 < 4096 ? (count + 255) / 256 : 4096);
+    if (dtype == BL_BF16)
+        BL_CUDA(bl_launch_dependent(scale_pairs_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16*)x,
+                                    wts, top, d, (__nv_bfloat16*)dst, count));
+    else
+        BL_CUDA(bl_launch_dependent(scale_pairs_kernel<float>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const float*)x, wts, top, d,
+                                    (float*)dst, count));
+    BL_CHECK_LAUNCH("bl_scale_pairs");
     return 0;
 }

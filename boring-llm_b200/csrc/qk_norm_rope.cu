@@ -10,6 +10,11 @@ namespace {
 
 constexpr int THREADS = 128;
 
+// Further options. norm_q / norm_k > 0: how many of a row's values the whole-row norms average over (heads that are padded
+// with zeros count their own values only). first: values of the same tokens that another layer projected, blended into this
+// layer's ones: heads of first_dv values, first_places apart; this layer's heads have dv values of their own (then zeros).
+struct BlBlendArgs { int norm_q, norm_k; const float* first; int ld_first, first_dv, first_places, dv; const void* lambda; int lambda_dtype; };
+
 __device__ __forceinline__ float block_sum(float v, float* part) {
     v = bl_warp_sum(v);
     __syncthreads();                                   // part may still be read from the call before
@@ -25,7 +30,7 @@ qk_norm_rope_write_kernel(const float* proj, int ld, int off_k, int off_v, const
                           const int* __restrict__ tok_req, const int* __restrict__ block_table, int max_pages,
                           const float* __restrict__ inv_freq, int rot_half, int pair_layout, TT* __restrict__ q_out,
                           TT* __restrict__ k_cache, TT* __restrict__ v_cache, int H, int KV, int dk, int dv, int page_size,
-                          int per_head, const float* __restrict__ q_head_scale) {
+                          int per_head, const float* __restrict__ q_head_scale, BlBlendArgs bl) {
     bl_pdl_trigger();
     bl_pdl_wait();
     extern __shared__ float cs[];                      // cos [rot_half], sin [rot_half], then (per_head) 1 / rms of each of the H + KV heads
@@ -52,12 +57,12 @@ qk_norm_rope_write_kernel(const float* proj, int ld, int off_k, int off_v, const
     } else if (qw) {
         float s = 0.f;
         for (int i = threadIdx.x; i < H * dk; i += THREADS) s += row[i] * row[i];
-        inv_q = 1.0f / sqrtf(block_sum(s, part) / (float)(H * dk) + eps);
+        inv_q = 1.0f / sqrtf(block_sum(s, part) / (float)(bl.norm_q > 0 ? bl.norm_q : H * dk) + eps);
     }
     if (kw && !per_head) {
         float s = 0.f;
         for (int i = threadIdx.x; i < KV * dk; i += THREADS) s += row[off_k + i] * row[off_k + i];
-        inv_k = 1.0f / sqrtf(block_sum(s, part) / (float)(KV * dk) + eps);
+        inv_k = 1.0f / sqrtf(block_sum(s, part) / (float)(bl.norm_k > 0 ? bl.norm_k : KV * dk) + eps);
     }
     __syncthreads();
     const int r = tok_req[t];
@@ -95,7 +100,17 @@ qk_norm_rope_write_kernel(const float* proj, int ld, int off_k, int off_v, const
     if (v_cache) {
         for (int e = threadIdx.x; e < KV * dv; e += THREADS) {
             const int g = e / dv, d = e % dv;
-            bl_store(v_cache + (((size_t)page * KV + g) * page_size + in_page) * dv + d, row[off_v + e]);
+            float v = row[off_v + e];
+            if (bl.first) {                            // v <- (1 - lambda) v + lambda first, channel by channel of the flat values
+                float f = 0.f;
+                if (d < bl.dv) {
+                    const int flat = g * bl.dv + d;
+                    f = bl.first[(size_t)t * bl.ld_first + (flat / bl.first_dv) * bl.first_places + flat % bl.first_dv];
+                }
+                const float lam = bl_load_any(bl.lambda, bl.lambda_dtype, 0);
+                v = (1.f - lam) * v + lam * f;
+            }
+            bl_store(v_cache + (((size_t)page * KV + g) * page_size + in_page) * dv + d, v);
         }
     }
 }
@@ -117,16 +132,34 @@ extern "C" int bl_qk_norm_rope_write_scope(const float* proj, int ld, int off_k,
                                            const int* tok_req, const int* block_table, int max_pages, const float* inv_freq,
                                            int rot_half, int pair_layout, void* q_out, void* k_cache, void* v_cache, int dtype, int T,
                                            int H, int KV, int dk, int dv, int page_size, const float* q_head_scale, void* stream) {
+    return bl_qk_norm_rope_write_ext(proj, ld, off_k, off_v, q_norm_w, qw_dtype, k_norm_w, kw_dtype, eps, per_head, positions, tok_req,
+                                     block_table, max_pages, inv_freq, rot_half, pair_layout, q_out, k_cache, v_cache, dtype, T, H,
+                                     KV, dk, dv, page_size, q_head_scale, 0, 0, nullptr, 0, 0, 0, 0, nullptr, 0, stream);
+}
+
+extern "C" int bl_qk_norm_rope_write_ext(const float* proj, int ld, int off_k, int off_v, const void* q_norm_w, int qw_dtype,
+                                         const void* k_norm_w, int kw_dtype, float eps, int per_head, const int* positions,
+                                         const int* tok_req, const int* block_table, int max_pages, const float* inv_freq,
+                                         int rot_half, int pair_layout, void* q_out, void* k_cache, void* v_cache, int dtype, int T,
+                                         int H, int KV, int dk, int dv, int page_size, const float* q_head_scale, int norm_q, int norm_k,
+                                         const float* v_first, int ld_first, int first_dv, int first_places, int dv_real, const void* lambda,
+                                         int lambda_dtype, void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || KV <= 0 || dk <= 0 || dv <= 0 || rot_half < 0 || 2 * rot_half > dk || page_size <= 0)
         BL_FAIL("bl_qk_norm_rope_write: bad sizes H=%d KV=%d dk=%d dv=%d rotated pairs=%d page=%d", H, KV, dk, dv, rot_half, page_size);
     if (ld < off_v + KV * dv || off_k < H * dk || off_v < off_k + KV * dk)
         BL_FAIL("bl_qk_norm_rope_write: columns q, k (%d), v (%d) do not fit rows of %d", off_k, off_v, ld);
+    if (norm_q < 0 || norm_q > H * dk || norm_k < 0 || norm_k > KV * dk)
+        BL_FAIL("bl_qk_norm_rope_write: norms over %d and %d values of rows of %d and %d", norm_q, norm_k, H * dk, KV * dk);
+    if (v_first && (!lambda || dv_real <= 0 || dv_real > dv || first_dv <= 0 || first_dv > first_places || KV * dv_real % first_dv != 0 ||
+                    ld_first < KV * dv_real / first_dv * first_places))
+        BL_FAIL("bl_qk_norm_rope_write: values of %d heads of %d cannot be blended with heads of %d in rows of %d", KV, dv_real, first_dv, ld_first);
+    const BlBlendArgs bl{norm_q, norm_k, v_first, ld_first, first_dv, first_places, dv_real, lambda, lambda_dtype};
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)(2 * rot_half + 1 + (per_head ? H + KV : 0)) * sizeof(float);
 #define BL_GO(TT) BL_CUDA(bl_launch_dependent(qk_norm_rope_write_kernel<TT>, dim3(T), dim3(THREADS), smem, s, proj, ld, off_k, off_v, \
         q_norm_w, qw_dtype, k_norm_w, kw_dtype, eps, positions, tok_req, block_table, max_pages, inv_freq, rot_half, pair_layout, \
-        (TT*)q_out, (TT*)k_cache, (TT*)v_cache, H, KV, dk, dv, page_size, per_head, q_head_scale))
+        (TT*)q_out, (TT*)k_cache, (TT*)v_cache, H, KV, dk, dv, page_size, per_head, q_head_scale, bl))
     if (dtype == BL_F32) BL_GO(float);
     else if (dtype == BL_BF16) BL_GO(__nv_bfloat16);
     else BL_FAIL("bl_qk_norm_rope_write: unknown dtype %d", dtype);

@@ -265,12 +265,13 @@ def qkv_rope_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], 
 def attention_plain(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, tok_req: torch.Tensor,
                     cu_q: torch.Tensor, ctx_len: torch.Tensor, block_table: torch.Tensor,
                     out: torch.Tensor, H: int, window: int, scale: float, sinks: Optional[torch.Tensor] = None,
-                    gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+                    gate: Optional[torch.Tensor] = None, softcap: float = 0.0, gate_dim: int = 0) -> None:
     """Paged causal grouped-query attention, one warp per (token, head). `softcap` c > 0: the scaled scores pass
     c * tanh(s / c) before the softmax. The values' head size may differ from the
     keys' (v_cache `[pages, kv heads, page, dv]`, out `[T, H * dv]`). `sinks` [H]: exp(sinks[h]) joins head h's softmax
     denominator (once, unscaled, no value). `gate` (32-bit, [T, >= H], rows contiguous, possibly a column range of a
-    wider matrix): head h of token t is multiplied by sigmoid(gate[t, h])."""
+    wider matrix): head h of token t is multiplied by sigmoid(gate[t, h]). `gate_dim` = dv: a logit
+    per channel instead, channel d of head h times sigmoid(gate[t, h * dv + d]) (every attention kernel has it)."""
     T = q.shape[0]
     n_pages, KV, page_size, dh = k_cache.shape
     dv = v_cache.shape[3]
@@ -278,17 +279,9 @@ def attention_plain(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     _need(v_cache, "v_cache", k_cache.dtype, (n_pages, KV, page_size, dv))
     _need(tok_req, "tok_req", torch.int32, (T,)); _need(cu_q, "cu_q", torch.int32); _need(ctx_len, "ctx_len", torch.int32)
     _need(block_table, "block_table", torch.int32); _need(out, "out", q.dtype, (T, H * dv))
-    if sinks is not None:
-        _need(sinks, "sinks", None, (H,))
-    ld_gate = 0
-    if gate is not None:
-        if not gate.is_cuda or gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < H:
-            raise KernelError("gate: must be 32-bit CUDA rows [T, >= H] with contiguous rows")
-        ld_gate = gate.stride(0)
     _call(_lib().bl_attention_plain_cap, _p(q), _p(k_cache), _p(v_cache), _dt(q), _p(tok_req), _p(cu_q),
           _p(ctx_len), _p(block_table), block_table.shape[1], _p(out), T, H, KV, dh, dv, page_size, window,
-          ctypes.c_float(scale), _p(sinks), _dt(sinks) if sinks is not None else 0, _p(gate), ld_gate, ctypes.c_float(softcap),
-          _stream())
+          ctypes.c_float(scale), *_tail(T, H, sinks, gate, gate_dim), gate_dim, ctypes.c_float(softcap), _stream())
 
 
 def argmax(logits: torch.Tensor, out_ids: torch.Tensor) -> None:
@@ -336,14 +329,15 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optio
           M, N, K, epilogue, _stream())
 
 
-def _tail(T: int, H: int, sinks: Optional[torch.Tensor], gate: Optional[torch.Tensor]):
-    """The arguments (sinks, their dtype, gate, its row stride) of the attention kernels' `_tail` entry points."""
+def _tail(T: int, H: int, sinks: Optional[torch.Tensor], gate: Optional[torch.Tensor], gate_dim: int = 0):
+    """The arguments (sinks, their dtype, gate, its row stride) of the attention kernels' `_tail` entry points. `gate_dim` n > 0:
+    the gate has a logit per channel, n for each head."""
     if sinks is not None:
         _need(sinks, "sinks", None, (H,))
     ld = 0
     if gate is not None:
-        if not gate.is_cuda or gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < H:
-            raise KernelError("gate: must be 32-bit CUDA rows [T, >= H] with contiguous rows")
+        if not gate.is_cuda or gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < H * max(1, gate_dim):
+            raise KernelError("gate: must be 32-bit CUDA rows [T, >= heads (times channels)] with contiguous rows")
         ld = gate.stride(0)
     return _p(sinks), _dt(sinks) if sinks is not None else 0, _p(gate), ld
 
@@ -354,7 +348,7 @@ def attention_mma_supported(dtype: torch.dtype, dh: int, page_size: int) -> bool
 
 def attention_prefill(q, k_cache, v_cache, cu_q, ctx_len, block_table, tiles, out, H: int, window: int,
                       scale: float, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                      softcap: float = 0.0) -> None:
+                      softcap: float = 0.0, gate_dim: int = 0) -> None:
     """Tensor-core attention for requests with several new tokens. tiles: int32 [n, 2] = (request, first token
     of a 64-token tile among the request's new tokens). `softcap` c > 0: scaled scores pass c tanh(s / c)."""
     T = q.shape[0]
@@ -363,10 +357,10 @@ def attention_prefill(q, k_cache, v_cache, cu_q, ctx_len, block_table, tiles, ou
     _need(v_cache, "v_cache", torch.bfloat16, k_cache.shape); _need(out, "out", torch.bfloat16, (T, H * dh))
     _need(cu_q, "cu_q", torch.int32); _need(ctx_len, "ctx_len", torch.int32); _need(block_table, "block_table", torch.int32)
     _need(tiles, "tiles", torch.int32)
-    if softcap > 0:
+    if softcap > 0 or gate_dim:
         _call(_lib().bl_attention_prefill_cap, _p(q), _p(k_cache), _p(v_cache), _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(tiles), tiles.shape[0], _p(out), H, KV, dh, page_size, window,
-          ctypes.c_float(scale), *_tail(T, H, sinks, gate), ctypes.c_float(softcap), _stream())
+          ctypes.c_float(scale), *_tail(T, H, sinks, gate, gate_dim), gate_dim, ctypes.c_float(softcap), _stream())
     elif sinks is None and gate is None:
         _call(_lib().bl_attention_prefill, _p(q), _p(k_cache), _p(v_cache), _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(tiles), tiles.shape[0], _p(out), H, KV, dh, page_size, window,
@@ -383,7 +377,7 @@ def attention_prefill_tc_supported(dtype: torch.dtype, dh: int, page_size: int) 
 
 def attention_prefill_tc(q, k_cache, v_cache, cu_q, ctx_len, block_table, tiles, out, H: int, window: int,
                          scale: float, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                         softcap: float = 0.0) -> None:
+                         softcap: float = 0.0, gate_dim: int = 0) -> None:
     """The tcgen05 form of `attention_prefill` (head size 64, pages of 16). tiles: int32 [n, 2] = (request,
     first token of a tile of 128 among the request's new tokens); the last entries are launched first. `softcap` c > 0:
     scaled scores pass c tanh(s / c) (a second build of the kernel; without a cap the kernel is the one it was)."""
@@ -393,10 +387,10 @@ def attention_prefill_tc(q, k_cache, v_cache, cu_q, ctx_len, block_table, tiles,
     _need(v_cache, "v_cache", torch.bfloat16, k_cache.shape); _need(out, "out", torch.bfloat16, (T, H * dh))
     _need(cu_q, "cu_q", torch.int32); _need(ctx_len, "ctx_len", torch.int32); _need(block_table, "block_table", torch.int32)
     _need(tiles, "tiles", torch.int32, (tiles.shape[0], 2))
-    if softcap > 0:
+    if softcap > 0 or gate_dim:
         _call(_lib().bl_attention_prefill_tc_cap, _p(q), _p(k_cache), _p(v_cache), _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(tiles), tiles.shape[0], _p(out), T, n_pages, H, KV, dh, page_size, window,
-          ctypes.c_float(scale), *_tail(T, H, sinks, gate), ctypes.c_float(softcap), _stream())
+          ctypes.c_float(scale), *_tail(T, H, sinks, gate, gate_dim), gate_dim, ctypes.c_float(softcap), _stream())
     elif sinks is None and gate is None:
         _call(_lib().bl_attention_prefill_tc, _p(q), _p(k_cache), _p(v_cache), _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(tiles), tiles.shape[0], _p(out), T, n_pages, H, KV, dh, page_size, window,
@@ -412,7 +406,7 @@ DECODE_CLUSTER_SPLITS = 16     # up to this many slices merge through distribute
 
 def attention_decode(q, k_cache, v_cache, cu_q, ctx_len, block_table, reqs, n_splits: int, out, H: int, window: int,
                      scale: float, scratch: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-                     gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+                     gate: Optional[torch.Tensor] = None, softcap: float = 0.0, gate_dim: int = 0) -> None:
     """Tensor-core attention for requests with one new token; `reqs` int32 [n] lists them. The keys of each are
     cut into `n_splits` slices. Up to `DECODE_CLUSTER_SPLITS` slices without `scratch`: the slices of a request are
     the blocks of a cluster and merge in shared memory. More slices, or a `scratch` tensor (float32,
@@ -442,10 +436,10 @@ def attention_decode(q, k_cache, v_cache, cu_q, ctx_len, block_table, reqs, n_sp
                 raise KernelError("attention_decode: its counters must exist before a capture (run the step once first)")
             # zero once; every launch leaves them at zero again
             counters = _decode_counters[q.device] = torch.zeros(max(n_counters, 4096), dtype=torch.int32, device=q.device)
-    if softcap > 0:
+    if softcap > 0 or gate_dim:
         _call(_lib().bl_attention_decode_cap, _p(q), _p(k_cache), _p(v_cache), _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(reqs), n, n_splits, _p(scratch if need else None), _p(counters), _p(out), H, KV, dh,
-          page_size, window, ctypes.c_float(scale), *_tail(T, H, sinks, gate), ctypes.c_float(softcap), _stream())
+          page_size, window, ctypes.c_float(scale), *_tail(T, H, sinks, gate, gate_dim), gate_dim, ctypes.c_float(softcap), _stream())
     elif sinks is None and gate is None:
         _call(_lib().bl_attention_decode, _p(q), _p(k_cache), _p(v_cache), _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(reqs), n, n_splits, _p(scratch if need else None), _p(counters), _p(out), H, KV, dh,
@@ -462,7 +456,7 @@ def attention_decode_tma_supported(dtype: torch.dtype, dh: int, page_size: int) 
 
 def attention_decode_tma(q, k_cache, v_cache, cu_q, ctx_len, block_table, reqs, n_splits: int, out, H: int, window: int,
                          scale: float, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                         softcap: float = 0.0) -> None:
+                         softcap: float = 0.0, gate_dim: int = 0) -> None:
     """`attention_decode` for head sizes 64 and 128 with keys and values streamed by TMA into per-warp rings and the
     query heads of a key/value head as the columns of the MMAs; 1 to `DECODE_CLUSTER_SPLITS` slices, which are the
     blocks of one cluster and send their partial rows to the blocks that finish them."""
@@ -479,10 +473,10 @@ def attention_decode_tma(q, k_cache, v_cache, cu_q, ctx_len, block_table, reqs, 
     G = H // KV
     blocks = n * KV * (-(-G // (8 if G <= 8 else 16))) * n_splits
     early = not (n_splits >= DECODE_TMA_LATE_CLUSTER and blocks > _sms())
-    if softcap > 0:                          # a cap on the scaled scores: a second build of the kernel
+    if softcap > 0 or gate_dim:              # (a cap on the scaled scores: a second build of the kernel)
         _call(_lib().bl_attention_decode_tma_cap, _p(q), _p(k_cache), _p(v_cache), n_pages, _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(reqs), n, n_splits, _p(out), H, KV, dh, page_size, window, ctypes.c_float(scale),
-          1 if early else 0, *_tail(T, H, sinks, gate), ctypes.c_float(softcap), _stream())
+          1 if early else 0, *_tail(T, H, sinks, gate, gate_dim), gate_dim, ctypes.c_float(softcap), _stream())
     elif sinks is None and gate is None:
         _call(_lib().bl_attention_decode_tma, _p(q), _p(k_cache), _p(v_cache), n_pages, _p(cu_q), _p(ctx_len), _p(block_table),
           block_table.shape[1], _p(reqs), n, n_splits, _p(out), H, KV, dh, page_size, window, ctypes.c_float(scale),
@@ -907,9 +901,13 @@ def activation(x: torch.Tensor, out: torch.Tensor, act: int) -> None:
 def qk_norm_rope_write(proj: torch.Tensor, off_k: int, off_v: int, q_norm_w: Optional[torch.Tensor],
                        k_norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor, tok_req: torch.Tensor,
                        block_table: torch.Tensor, inv_freq: torch.Tensor, rot_half: int, pair_layout: int, q_out: torch.Tensor,
-                       k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], H: int, KV: int, dk: int, dv: int) -> None:
+                       k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], H: int, KV: int, dk: int, dv: int,
+                       norm_q: int = 0, norm_k: int = 0, blend=None) -> None:
     """From a token's joined projections (32-bit rows: q first, k from column off_k, v from off_v): RMS norm over the
-    whole q row and the whole k row (weights None: no norm), rotation, q out, k and v into the request's pages."""
+    whole q row and the whole k row (weights None: no norm), rotation, q out, k and v into the request's pages. `norm_q` / `norm_k`
+    > 0: how many of a row's values the norms average over (heads padded with zeros). `blend` = (values [T, >= ..] of the same
+    tokens in 32-bit, their heads' size, the places from head to head, this layer's own value head size, lambda [1]): the
+    cached values are (1 - lambda) v + lambda * those, matched channel by channel over the flat row."""
     T = proj.shape[0]
     ld = _rows32(proj, "proj", T, off_v + KV * dv)
     _need(positions, "positions", torch.int32, (T,)); _need(tok_req, "tok_req", torch.int32, (T,))
@@ -927,10 +925,20 @@ def qk_norm_rope_write(proj: torch.Tensor, off_k: int, off_v: int, q_norm_w: Opt
         if tuple(k_cache.shape[1:]) != (KV, k_cache.shape[2], dk) or tuple(v_cache.shape) != (k_cache.shape[0], KV, k_cache.shape[2], dv):
             raise KernelError(f"caches {tuple(k_cache.shape)} / {tuple(v_cache.shape)} do not hold {KV} heads of {dk} / {dv}")
         page_size = k_cache.shape[2]
-    _call(_lib().bl_qk_norm_rope_write, _p(proj), ld, off_k, off_v, _p(q_norm_w), _dt(q_norm_w) if q_norm_w is not None else 0,
-          _p(k_norm_w), _dt(k_norm_w) if k_norm_w is not None else 0, ctypes.c_float(eps), _p(positions), _p(tok_req),
-          _p(block_table), block_table.shape[1], _p(inv_freq), rot_half, pair_layout, _p(q_out), _p(k_cache), _p(v_cache),
-          _dt(q_out), T, H, KV, dk, dv, page_size, _stream())
+    if not (norm_q or norm_k or blend):
+        _call(_lib().bl_qk_norm_rope_write, _p(proj), ld, off_k, off_v, _p(q_norm_w), _dt(q_norm_w) if q_norm_w is not None else 0,
+              _p(k_norm_w), _dt(k_norm_w) if k_norm_w is not None else 0, ctypes.c_float(eps), _p(positions), _p(tok_req),
+              _p(block_table), block_table.shape[1], _p(inv_freq), rot_half, pair_layout, _p(q_out), _p(k_cache), _p(v_cache),
+              _dt(q_out), T, H, KV, dk, dv, page_size, _stream())
+        return
+    first, first_dv, first_places, dv_real, lam = blend if blend is not None else (None, 0, 0, 0, None)
+    if first is not None:
+        _rows32(first, "the other layer's values", T, KV * dv_real // first_dv * first_places)
+        _need(lam, "lambda", None, (1,))
+    _call(_lib().bl_qk_norm_rope_write_ext, _p(proj), ld, off_k, off_v, _p(q_norm_w), _vec_dt(q_norm_w), _p(k_norm_w), _vec_dt(k_norm_w),
+          ctypes.c_float(eps), 0, _p(positions), _p(tok_req), _p(block_table), block_table.shape[1], _p(inv_freq), rot_half, pair_layout,
+          _p(q_out), _p(k_cache), _p(v_cache), _dt(q_out), T, H, KV, dk, dv, page_size, _p(None), norm_q, norm_k, _p(first),
+          first.stride(0) if first is not None else 0, first_dv, first_places, dv_real, _p(lam), _vec_dt(lam), _stream())
 
 
 def gemm_plain_decay(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], coef: torch.Tensor, group: int, sign: float,
@@ -1334,13 +1342,16 @@ def expert_gemm_plain(x: torch.Tensor, x_div: int, w: torch.Tensor, ids: torch.T
           P, N, K, epilogue, _p(act), w.shape[0], _stream())
 
 
-def moe_combine(y: torch.Tensor, wts: torch.Tensor, out: torch.Tensor, add: bool = False, ids: Optional[torch.Tensor] = None,
-                n_real: int = 0, x: Optional[torch.Tensor] = None) -> None:
+def moe_combine(y: torch.Tensor, wts: Optional[torch.Tensor], out: torch.Tensor, add: bool = False, ids: Optional[torch.Tensor] = None,
+                n_real: int = 0, x: Optional[torch.Tensor] = None, top: int = 0) -> None:
     """out[t] = sum_k wts[t, k] * y[t * top + k], k ascending (32-bit); with `add` the sum is added to out. With `ids`, a pair
-    whose expert number is `n_real` or more is an identity expert and contributes x[t] (the token's input row) instead."""
-    T, top = wts.shape
-    d = out.shape[1]
-    _need(y, "y", torch.float32, (T * top, d)); _need(wts, "wts", torch.float32); _need(out, "out", torch.float32, (T, d))
+    whose expert number is `n_real` or more is an identity expert and contributes x[t] (the token's input row) instead. wts None:
+    ones (then `top` says how many rows a token has)."""
+    T, d = out.shape
+    if wts is not None:
+        top = wts.shape[1]
+        _need(wts, "wts", torch.float32, (T, top))
+    _need(y, "y", torch.float32, (T * top, d)); _need(out, "out", torch.float32, (T, d))
     if ids is not None:
         _need(ids, "ids", torch.int32, (T, top)); _need(x, "x", None, (T, d))
     _call(_lib().bl_moe_combine_some, _p(y), _p(wts), _p(out), T, top, d, 1 if add else 0, _p(ids), n_real, _p(x),
@@ -1371,10 +1382,20 @@ def moe_plan(ids: torch.Tensor, n_experts: int):
     return pos, row_src, tile_expert
 
 
-def gather_rows(x: torch.Tensor, row_src: torch.Tensor, div: int, out: torch.Tensor) -> None:
-    """out[row] = x[row_src[row] // div] (zeros where row_src is negative); bfloat16 rows of a multiple of 8 values."""
+def gather_rows(x: torch.Tensor, row_src: torch.Tensor, div: int, out: torch.Tensor, wts: Optional[torch.Tensor] = None) -> None:
+    """out[row] = x[row_src[row] // div] (zeros where row_src is negative); bfloat16 rows of a multiple of 8 values. `wts` (32-bit,
+    one per pair): times wts[row_src[row]]."""
+    if wts is not None:
+        _need(wts, "wts", torch.float32, (x.shape[0], div))
     _need(x, "x", torch.bfloat16); _need(out, "out", torch.bfloat16, (row_src.numel(), x.shape[1])); _need(row_src, "row_src", torch.int32)
-    _call(_lib().bl_gather_rows, _p(x), _p(row_src), div, _p(out), out.shape[0], x.shape[1], _stream())
+    _call(_lib().bl_gather_rows_weighted, _p(x), _p(row_src), div, _p(wts), _p(out), out.shape[0], x.shape[1], _stream())
+
+
+def scale_pairs(x: torch.Tensor, wts: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t * top + k] = x[t] * wts[t, k] (wts 32-bit [T, top]; x and out of one dtype): what a pair's expert reads."""
+    T, top = wts.shape
+    _need(x, "x", None, (T, x.shape[1])); _need(wts, "wts", torch.float32); _need(out, "out", x.dtype, (T * top, x.shape[1]))
+    _call(_lib().bl_scale_pairs, _p(x), _dt(x), _p(wts), T, top, x.shape[1], _p(out), _stream())
 
 
 def gemm_grouped(x: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, out: torch.Tensor, epilogue: int = EPI_NONE,
@@ -1394,13 +1415,15 @@ def gemm_grouped(x: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, ou
     _call(_lib().bl_gemm_tc_grouped, _p(x), _p(w), _p(out), _dt(out), M, N, K, epilogue, E, _p(tile_expert), _p(act), _stream())
 
 
-def moe_combine_rows(y: torch.Tensor, pos: torch.Tensor, wts: torch.Tensor, out: torch.Tensor, add: bool = False,
+def moe_combine_rows(y: torch.Tensor, pos: torch.Tensor, wts: Optional[torch.Tensor], out: torch.Tensor, add: bool = False,
                      x: Optional[torch.Tensor] = None) -> None:
     """out[t] = sum_k wts[t, k] * y[pos[t * top + k]], k ascending (32-bit); with `add` the sum is added to out. A pair without
-    a row (pos < 0: an identity expert, see `moe_plan`) contributes x[t], the token's input row."""
-    T, top = wts.shape
-    d = out.shape[1]
-    _need(y, "y", torch.float32); _need(pos, "pos", torch.int32, (T * top,)); _need(wts, "wts", torch.float32); _need(out, "out", torch.float32, (T, d))
+    a row (pos < 0: an identity expert, see `moe_plan`) contributes x[t], the token's input row. wts None: ones."""
+    T, d = out.shape
+    top = pos.numel() // T
+    if wts is not None:
+        _need(wts, "wts", torch.float32, (T, top))
+    _need(y, "y", torch.float32); _need(pos, "pos", torch.int32, (T * top,)); _need(out, "out", torch.float32, (T, d))
     if y.shape[1] != d:
         raise KernelError("moe_combine_rows: y and out differ in width")
     if x is not None:
@@ -1767,3 +1790,62 @@ def xielu(x: torch.Tensor, out: torch.Tensor, args: torch.Tensor) -> None:
     if out.stride(1) != 1:
         raise KernelError("xielu: out must have contiguous rows")
     _call(_lib().bl_xielu, _p(x), ctypes.c_longlong(ld), _p(out), _dt(out), ctypes.c_longlong(out.stride(0)), rows, cols, _p(args), _stream())
+
+
+# ---- a residual of several streams, an embedding of token pairs ------------------------------------------------------
+HYPER_MAX_STREAMS = 16
+
+
+def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, tok_req: torch.Tensor,
+                cu_q: torch.Tensor, slots: torch.Tensor, prev_tokens: torch.Tensor, mul_prev: int, mul_cur: int, out: torch.Tensor) -> None:
+    """out[t] = table[ids[t]] + pairs[(previous token * mul_prev + ids[t] * mul_cur) mod buckets], 32-bit; pairs [buckets + 1, d],
+    its last row for a sequence's first token. prev_tokens (int32, one per slot) carries each request's last token from step to step."""
+    T = ids.shape[0]
+    d = table.shape[1]
+    _need(table, "table"); _need(pairs, "pairs", table.dtype, (pairs.shape[0], d)); _need(ids, "ids", torch.int32, (T,))
+    _need(positions, "positions", torch.int32, (T,)); _need(tok_req, "tok_req", torch.int32, (T,)); _need(cu_q, "cu_q", torch.int32)
+    _need(slots, "slots", torch.int32); _need(prev_tokens, "prev_tokens", torch.int32); _need(out, "out", torch.float32, (T, d))
+    _call(_lib().bl_embed_pairs, _p(table), _p(pairs), _dt(table), _p(ids), _p(positions), _p(tok_req), _p(cu_q), _p(slots), _p(prev_tokens),
+          ctypes.c_longlong(mul_prev), ctypes.c_longlong(mul_cur), ctypes.c_longlong(pairs.shape[0] - 1), _p(out), T, d, _stream())
+
+
+def hyper_step(x: torch.Tensor, n: int, x_out: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None,
+               y: Optional[torch.Tensor] = None, y_pos: Optional[torch.Tensor] = None, y_wts: Optional[torch.Tensor] = None, top: int = 1,
+               read: Optional[torch.Tensor] = None, norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
+               h: Optional[torch.Tensor] = None, row_idx: Optional[torch.Tensor] = None) -> None:
+    """One pass over a residual of n streams: x [n, T, d], or [T, d] while all streams are the same rows.
+
+    `write` (32-bit, n + n * n numbers: b, then M [from, to]): x'_t = sum_s M[s, t] x_s + b[t] y, into x_out [n, T, d] (x itself: in
+    place; None: not stored); y [T, d], or the rows of routed pairs: token t's result is sum_k y_wts[t, k] (None: 1) *
+    y[y_pos[t * top + k]] (y_pos None: row t * top + k). `h` [rows, d]: sum_s read[s] x'_s (read None: the plain sum) of tokens
+    row_idx (None: all), with `norm_w` divided by its root mean square and multiplied by the weight."""
+    T, d = x.shape[-2:]
+    _need(x, "x", torch.float32)
+    if x.dim() == 3 and x.shape[0] != n:
+        raise KernelError(f"x: {x.shape[0]} streams, {n} expected")
+    if x_out is not None:
+        _need(x_out, "x_out", torch.float32, (n, T, d))
+    if write is not None:
+        _need(write, "write", torch.float32, (n + n * n,)); _need(y, "y", torch.float32)
+        if y.shape[1] != d or (y_pos is None and y.shape[0] != T * top):
+            raise KernelError(f"y: {tuple(y.shape)} does not hold {top} rows of {d} for each of {T} tokens")
+        if y_pos is not None:
+            _need(y_pos, "y_pos", torch.int32, (T * top,))
+        if y_wts is not None:
+            _need(y_wts, "y_wts", torch.float32, (T, top))
+    if read is not None:
+        _need(read, "read", torch.float32, (n,))
+    rows = T
+    if row_idx is not None:
+        _need(row_idx, "row_idx", torch.int32)
+        if x_out is not None:
+            raise KernelError("hyper_step: chosen rows are read, not written back")
+        rows = row_idx.shape[0]
+    if norm_w is not None:
+        _need(norm_w, "norm_w", None, (d,))
+    if h is not None:
+        _need(h, "h", None, (rows, d))
+    ll = ctypes.c_longlong
+    _call(_lib().bl_hyper_step, _p(x), ll(T * d if x.dim() == 3 else 0), _p(x_out), ll(T * d), n, _p(write), _p(y), _p(y_pos), _p(y_wts),
+          top, _p(read), _p(norm_w), _vec_dt(norm_w), ctypes.c_float(eps), _p(h), _dt(h) if h is not None else 0, _p(row_idx), rows, d,
+          _stream())

@@ -9,9 +9,10 @@ from .recurrent import (GatedLinearAttention, ChannelDeltaRule, MatrixMemory, Sh
 from .latent import LatentAttention
 from .feedforward import (FeedForward, SwiGLU, DenseMLP, RoutedExperts, GluMLP, SumFeedForward, TableExperts,
                           RowGatedFeedForward)
-from .block import PreNormBlock, GatedSandwichBlock, ResidualGate, PostNormBlock, ParallelBlock
+from .block import PreNormBlock, GatedSandwichBlock, ResidualGate, PostNormBlock, ParallelBlock, HyperBlock
 from .depth import DepthWeightedAverage, StreamReentry
-from .embedding import Embedding, OutputHead
+from .streams import HyperConnection, StreamResidual
+from .embedding import Embedding, PairEmbedding, OutputHead
 from .model import DecoderModel, LayerCall
 
 __all__ = ["Part", "StepContext", "StepPlan", "to_device_matrix", "to_device_vector", "linear", "RMSNorm",
@@ -20,4 +21,4 @@ __all__ = ["Part", "StepContext", "StepPlan", "to_device_matrix", "to_device_vec
            "ChunkedTalkingAttention", "ParallelMixers", "MatrixMemory", "ShiftedDecayRecurrence", "RoutedExperts", "PostNormBlock",
            "DepthWeightedAverage", "LatentAttention", "GluMLP", "SumFeedForward", "TableExperts",
            "MixedScoreAttention", "distance_slopes", "StreamReentry", "Retention", "StateSpaceDuality", "RowGatedFeedForward", "ParallelBlock",
-           "Embedding", "OutputHead", "DecoderModel", "LayerCall"]
+           "HyperBlock", "HyperConnection", "StreamResidual", "Embedding", "PairEmbedding", "OutputHead", "DecoderModel", "LayerCall"]

@@ -67,18 +67,19 @@ def attention_plan(q_lens, ctx_lens, filler=None) -> StepPlan:
 
 
 def paged_attention(ctx, q, k_cache, v_cache, table, out, H: int, KV: int, dh: int, window: int, scale: float,
-                    sinks=None, gate=None, softcap: float = 0.0) -> None:
+                    sinks=None, gate=None, softcap: float = 0.0, gate_dim: int = 0) -> None:
     """Causal attention of the step's tokens over the paged cache. Tensor-core kernels for bfloat16 where they are built
     (pages of 16, common head sizes, values of the keys' head size): one launch for the requests with several new tokens
     (the tcgen05 kernel for head sizes 64 and 128 when the step has many of them), one for those with a single token.
     Otherwise, and always in float32, the plain kernel. Which requests those are comes from the step's plan
     (`attention_plan`). `sinks` [H] and `gate` (32-bit logits [T, >= H]) are what may follow the softmax: a score per
-    head that joins the denominator, a sigmoid per (token, head) on the output. `softcap` c > 0: scaled scores pass
+    head that joins the denominator, a sigmoid per (token, head) on the output, or, with `gate_dim` = dv and logits [T, >= H * dv],
+    per (token, head, channel). `softcap` c > 0: scaled scores pass
     c tanh(s / c) before the softmax (every attention kernel has it)."""
     dv = v_cache.shape[3]
-    if not (ctx.fast and dv == dh and ops.attention_mma_supported(q.dtype, dh, k_cache.shape[2])):
+    if not (ctx.fast and dv == dh and scale > 0 and ops.attention_mma_supported(q.dtype, dh, k_cache.shape[2])):
         ops.attention_plain(q, k_cache, v_cache, ctx.tok_req, ctx.cu_q, ctx.ctx_len, table, out, H, window, scale, sinks, gate,
-                            softcap=softcap)
+                            softcap=softcap, gate_dim=gate_dim)
         return
     plan = ctx.plans.get(PLAN_KEY)
     if plan is None:                                 # a step put together without asking the parts: plan it now
@@ -89,10 +90,10 @@ def paged_attention(ctx, q, k_cache, v_cache, table, out, H: int, KV: int, dh: i
     if tiles64.shape[0]:
         if tiles128.shape[0] and ops.attention_prefill_tc_supported(q.dtype, dh, k_cache.shape[2]):
             ops.attention_prefill_tc(q, k_cache, v_cache, ctx.cu_q, ctx.ctx_len, table, tiles128, out, H, window, scale, sinks, gate,
-                                     softcap=softcap)
+                                     softcap=softcap, gate_dim=gate_dim)
         else:
             ops.attention_prefill(q, k_cache, v_cache, ctx.cu_q, ctx.ctx_len, table, tiles64, out, H, window, scale, sinks, gate,
-                                  softcap=softcap)
+                                  softcap=softcap, gate_dim=gate_dim)
     n = singles.shape[0]
     if n:
         # as many slices of the keys as fill the device once (the kernel knows how many of its blocks fit)
@@ -104,13 +105,13 @@ def paged_attention(ctx, q, k_cache, v_cache, table, out, H: int, KV: int, dh: i
             # head sizes 64 and 128: the TMA-fed kernel, which knows how many slices pay for this many requests
             n_splits = ops.attention_decode_tma_splits(n, KV, G, dh, longest)
             ops.attention_decode_tma(q, k_cache, v_cache, ctx.cu_q, ctx.ctx_len, table, singles, n_splits, out, H, window, scale,
-                                     sinks, gate, softcap=softcap)
+                                     sinks, gate, softcap=softcap, gate_dim=gate_dim)
             return
         groups = KV * (-(-G // 16))
         resident = ops.attention_decode_resident_blocks(dh)
         n_splits = max(1, min(-(-longest // 64), resident // (n * groups), DECODE_MAX_SPLITS))
         ops.attention_decode(q, k_cache, v_cache, ctx.cu_q, ctx.ctx_len, table, singles, n_splits, out, H, window, scale,
-                             sinks=sinks, gate=gate, softcap=softcap)
+                             sinks=sinks, gate=gate, softcap=softcap, gate_dim=gate_dim)
 
 
 class Mixer(Part):
@@ -273,6 +274,25 @@ class GQAAttention(Mixer):
     def attend(self, ctx, q, k_cache, v_cache, table, out):
         paged_attention(ctx, q, k_cache, v_cache, table, out, self.H, self.KV, self.dh, self.window, self.scale)
 
+BUILT_HEAD_SIZES = (16, 32, 48, 64, 96, 128)        # head sizes of the tensor-core attention kernels
+
+
+def padded_head(dk: int, dv: int) -> int:
+    """The places that heads of dk query/key and dv value channels take when both are padded with zeros to one size that the
+    tensor-core kernels have (0: there is none, they stay as they are)."""
+    return next((n for n in BUILT_HEAD_SIZES if n >= max(dk, dv)), 0)
+
+
+def _pad_head_rows(w, heads: int, places: int):
+    """w [heads * n, ...] with every head's n rows followed by zero rows up to `places`."""
+    n = w.shape[0] // heads
+    if n == places:
+        return w
+    out = w.new_zeros((heads, places) + tuple(w.shape[1:]))
+    out[:, :n] = w.reshape((heads, n) + tuple(w.shape[1:]))
+    return out.reshape((heads * places,) + tuple(w.shape[1:]))
+
+
 class GatedSinkAttention(Mixer):
     """Causal grouped-query attention over the paged cache with the options of newer designs, each a constructor
     argument:
@@ -285,7 +305,13 @@ class GatedSinkAttention(Mixer):
     * `sink=True`: a learned score per head whose exponential joins the softmax's denominator once, unscaled, with no
       key and no value;
     * `out_gate=True`: head h's output is multiplied by sigmoid(h . Wg^T)[h], one number per token and head, read from
-      the same rows as the projections;
+      the same rows as the projections; "channel": Wg has H * dv rows and every channel of the concatenated heads has a
+      sigmoid of its own;
+    * `value_mix`: layers of a model that blend their values with those of the first such layer, for the same tokens:
+      "first": this is that layer; "follow": v <- (1 - lambda) v + lambda v_first with a learned number `vmix`, in 32-bit, as the
+      values are cached (both layers' values, heads side by side, have one width; None: no blending);
+    * `pad_heads=True`: heads are padded with zeros (in the weights, at load) to one size for keys and values that the
+      tensor-core kernels are built for, where there is one; nothing of the result changes;
     * `qkv_bias=True` / `out_bias=True`: a bias on q, k and v, added in the joined product, and one on the output projection;
     * `softcap` c > 0: score <- c tanh(score / c) on the scaled score, before the softmax.
 
@@ -296,11 +322,14 @@ class GatedSinkAttention(Mixer):
 
     def __init__(self, dim: int, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: Optional[int],
                  rotary: Optional[RotaryTable], names: Dict[str, str], window: int = 0, scale: Optional[float] = None,
-                 qk_norm: Optional[str] = None, qk_norm_eps: float = 1e-6, sink: bool = False, out_gate: bool = False,
-                 qkv_bias: bool = False, out_bias: bool = False, softcap: float = 0.0):
+                 qk_norm: Optional[str] = None, qk_norm_eps: float = 1e-6, sink: bool = False, out_gate=False,
+                 qkv_bias: bool = False, out_bias: bool = False, softcap: float = 0.0, value_mix: Optional[str] = None,
+                 pad_heads: bool = False):
         super().__init__(names)
         if n_heads % n_kv_heads != 0:
             raise ValueError(f"{n_heads} query heads cannot share {n_kv_heads} key/value heads")
+        if out_gate not in (False, True, "head", "channel") or value_mix not in (None, "first", "follow"):
+            raise ValueError(f"GatedSinkAttention: out_gate {out_gate!r}, value_mix {value_mix!r}")
         if softcap < 0:
             raise ValueError(f"a cap on the scores must not be negative, got {softcap}")
         self.qkv_bias, self.out_bias, self.softcap = bool(qkv_bias), bool(out_bias), float(softcap)
@@ -313,11 +342,16 @@ class GatedSinkAttention(Mixer):
         self.window = int(window)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
         self.qk_norm, self.qk_norm_eps, self.has_sink, self.out_gate = qk_norm, float(qk_norm_eps), bool(sink), bool(out_gate)
-        self.off_k = self.H * self.dk
-        self.off_v = self.off_k + self.KV * self.dk
-        self.off_g = self.off_v + self.KV * self.dv
-        self.n_in = self.off_g + (self.H if self.out_gate else 0)
-        self.w_in = self.wo = self.q_norm = self.k_norm = self.sinks = None
+        self.channel_gate, self.value_mix = out_gate == "channel", value_mix
+        # the places a head takes in the joined product, in the cache and in the output (pk = dk and pv = dv without padding)
+        places = padded_head(self.dk, self.dv) if pad_heads else 0
+        self.pk, self.pv = places or self.dk, places or self.dv
+        self.off_k = self.H * self.pk
+        self.off_v = self.off_k + self.KV * self.pk
+        self.off_g = self.off_v + self.KV * self.pv
+        self.n_gate = (self.H * self.pv if self.channel_gate else self.H) if self.out_gate else 0
+        self.n_in = self.off_g + self.n_gate
+        self.w_in = self.wo = self.q_norm = self.k_norm = self.sinks = self.vmix = None
 
     def local_specs(self):
         s = {"wq": TensorSpec((self.H * self.dk, self.dim), MATRIX), "wk": TensorSpec((self.KV * self.dk, self.dim), MATRIX),
@@ -328,7 +362,9 @@ class GatedSinkAttention(Mixer):
         if self.has_sink:
             s["sink"] = TensorSpec((self.H,), BIAS)
         if self.out_gate:
-            s["wg"] = TensorSpec((self.H, self.dim), MATRIX)
+            s["wg"] = TensorSpec((self.H * self.dv if self.channel_gate else self.H, self.dim), MATRIX)
+        if self.value_mix == "follow":
+            s["vmix"] = TensorSpec((), BIAS)
         if self.qkv_bias:
             s.update({"bq": TensorSpec((self.H * self.dk,), BIAS), "bk": TensorSpec((self.KV * self.dk,), BIAS),
                       "bv": TensorSpec((self.KV * self.dv,), BIAS)})
@@ -337,26 +373,45 @@ class GatedSinkAttention(Mixer):
         return s
 
     def place(self, local, dtype, device):
-        joined = [local["wq"], local["wk"], local["wv"]] + ([local["wg"]] if self.out_gate else [])
+        pad = lambda t, heads, places: _pad_head_rows(t, heads, places)
+        layout = (("q", self.H, self.pk), ("k", self.KV, self.pk), ("v", self.KV, self.pv))
+        joined = [pad(local["w" + n], heads, places) for n, heads, places in layout]
+        if self.out_gate:
+            joined.append(pad(local["wg"], self.H, self.pv) if self.channel_gate else local["wg"])
         self.w_in = to_device_matrix(torch.cat(joined, dim=0), dtype, device)
-        self.wo = to_device_matrix(local["wo"], dtype, device)
+        self.wo = to_device_matrix(pad(local["wo"].t().contiguous(), self.H, self.pv).t(), dtype, device)
         if self.qkv_bias:                        # the gate's logits (further columns of the joined product) have none
-            b = [local[n].to(torch.float32) for n in ("bq", "bk", "bv")] + ([torch.zeros(self.H)] if self.out_gate else [])
+            b = [pad(local["b" + n].to(torch.float32), heads, places) for n, heads, places in layout]
+            b += [b[0].new_zeros(self.n_gate)] if self.out_gate else []
             self.b_in = torch.cat(b, dim=0).to(device).contiguous()
         if self.out_bias:
             self.bo = to_device_vector(local["bo"], dtype, device)
         if self.qk_norm:
-            self.q_norm = to_device_vector(local["q_norm"], dtype, device)
-            self.k_norm = to_device_vector(local["k_norm"], dtype, device)
+            self.q_norm = to_device_vector(pad(local["q_norm"], self.H, self.pk), dtype, device)
+            self.k_norm = to_device_vector(pad(local["k_norm"], self.KV, self.pk), dtype, device)
+        if self.value_mix == "follow":
+            self.vmix = to_device_vector(local["vmix"].reshape(1), dtype, device)
         if self.has_sink:
             self.sinks = to_device_vector(local["sink"], dtype, device)
         self.rotary.to(device)
 
     def cache_spec(self):
-        return PagedKVSpec(self.KV, self.dk, self.window, 0 if self.dv == self.dk else self.dv)
+        return PagedKVSpec(self.KV, self.pk, self.window, 0 if self.pv == self.pk else self.pv)
 
     def plan_step(self, q_lens, ctx_lens, filler=None):
         return PLAN_KEY, attention_plan(q_lens, ctx_lens, filler)
+
+    def _blend(self, ctx, proj):
+        """What the cached values are blended with: the first layer's projected values of this step's tokens, which that layer
+        leaves in the step's memo (32-bit columns of its joined product)."""
+        if self.value_mix == "first":
+            ctx.memo["first values"] = (proj[:, self.off_v:self.off_v + self.KV * self.pv], self.dv, self.pv, self.KV * self.dv)
+        if self.value_mix != "follow":
+            return None
+        values, dv, places, width = ctx.memo["first values"]
+        if width != self.KV * self.dv:
+            raise ValueError(f"values of {self.KV} heads of {self.dv} cannot be blended with rows of {width}")
+        return values, dv, places, self.dv, self.vmix
 
     def _run(self, ctx, h, out, cache_layer, write_cache, epilogue):
         T = h.shape[0]
@@ -364,13 +419,14 @@ class GatedSinkAttention(Mixer):
         proj = ctx.empty((T, self.w_in.shape[0]), torch.float32)
         linear(ctx, h, self.w_in, proj, self._bias_in(), EPI_BIAS if self.qkv_bias else EPI_NONE)
         self._joined(proj)
-        q = ctx.empty((T, self.H * self.dk))
+        q = ctx.empty((T, self.H * self.pk))
         ops.qk_norm_rope_write(proj, self.off_k, self.off_v, self.q_norm, self.k_norm, self.qk_norm_eps, ctx.positions,
                                ctx.tok_req, table, self.rotary.inv_freq, self.rotary.rot_half, self.rotary.pair_layout, q,
                                k_cache if write_cache else None, v_cache if write_cache else None, self.H, self.KV,
-                               self.dk, self.dv)
-        attn = ctx.empty((T, self.H * self.dv))
-        gate = proj[:, self.off_g:self.off_g + self.H] if self.out_gate else None
+                               self.pk, self.pv, norm_q=self.H * self.dk if self.pk != self.dk else 0,
+                               norm_k=self.KV * self.dk if self.pk != self.dk else 0, blend=self._blend(ctx, proj))
+        attn = ctx.empty((T, self.H * self.pv))
+        gate = proj[:, self.off_g:self.off_g + self.n_gate] if self.out_gate else None
         self.attend(ctx, q, k_cache, v_cache, table, attn, gate)
         if self.out_bias:
             if epilogue == EPI_RESIDUAL:
@@ -396,8 +452,8 @@ class GatedSinkAttention(Mixer):
         self._run(ctx, h, out, cache_layer, write_cache, EPI_NONE)
 
     def attend(self, ctx, q, k_cache, v_cache, table, out, gate):
-        paged_attention(ctx, q, k_cache, v_cache, table, out, self.H, self.KV, self.dk, self.window, self.scale, self.sinks, gate,
-                        softcap=self.softcap)
+        paged_attention(ctx, q, k_cache, v_cache, table, out, self.H, self.KV, self.pk, self.window, self.scale, self.sinks, gate,
+                        softcap=self.softcap, gate_dim=self.pv if self.channel_gate else 0)
 
 
 class ChunkedTalkingAttention(Mixer):

@@ -214,6 +214,51 @@ class GatedSandwichBlock(Part):
         return None
 
 
+class HyperBlock(Part):
+    """Pre-norm sublayers on a residual of several streams (`parts.streams`):
+
+        y = mixer(norm1(in1 . streams)) goes back through connection 1;   y = ffn(norm2(in2 . streams)) through connection 2
+
+    (a block without a feed-forward has only the first). `forward` takes the step's `StreamResidual` in the place of the stream.
+    The sublayers write their results instead of adding them; routed experts leave the sum over a token's experts to the
+    pass that writes back."""
+
+    def __init__(self, mixer_norm, mixer, mixer_connection, ffn_norm=None, ffn=None, ffn_connection=None):
+        super().__init__()
+        if (ffn is None) != (ffn_norm is None) or (ffn is None) != (ffn_connection is None):
+            raise ValueError("HyperBlock: a feed-forward, its norm and its connection come together")
+        self.mixer_norm, self.mixer, self.mixer_connection = mixer_norm, mixer, mixer_connection
+        self.ffn_norm, self.ffn, self.ffn_connection = ffn_norm, ffn, ffn_connection
+
+    def children(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_connection, self.ffn_norm, self.ffn, self.ffn_connection)
+                     if p is not None)
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    @property
+    def graph_safe(self) -> bool:
+        return bool(getattr(self.mixer, "graph_safe", False) and (self.ffn is None or getattr(self.ffn, "graph_safe", False)))
+
+    def forward(self, ctx, streams, cache_layer, write_cache: bool = True) -> None:
+        ctx.next_norm = None                     # no product adds into a stream, so none begins a norm
+        h = streams.read(ctx, self.mixer_connection, self.mixer_norm)
+        y = ctx.empty(streams.shape, torch.float32)
+        self.mixer.mix(ctx, h, y, cache_layer, write_cache)
+        streams.write(self.mixer_connection, y)
+        if self.ffn is None:
+            return
+        h = streams.read(ctx, self.ffn_connection, self.ffn_norm)
+        pairs = self.ffn.apply_pairs(ctx, h) if hasattr(self.ffn, "apply_pairs") else None
+        if pairs is not None:
+            streams.write(self.ffn_connection, *pairs, top=self.ffn.top)
+            return
+        y = ctx.empty(streams.shape, torch.float32)
+        self.ffn.apply(ctx, h, y)
+        streams.write(self.ffn_connection, y)
+
+
 class PostNormBlock(Part):
     """The norm stands BEHIND each sublayer and the sublayers read the residual stream itself:
 

@@ -5,6 +5,7 @@ from typing import Dict, Optional
 
 import torch
 
+from ..cache import StateSpec
 from ..kernels import ops
 from ..weights import TensorSpec, MATRIX
 from .base import Part, to_device_matrix
@@ -32,6 +33,29 @@ class Embedding(Part):
     def forward(self, ctx, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         x = ctx.empty((ctx.T, self.dim), torch.float32) if out is None else out
         ops.embed(self.table, ctx.token_ids, x, self.scale)
+        return x
+
+
+class PairEmbedding(Part):
+    """x[t] = table[token] + pairs[(previous token * mul_prev + token * mul_cur) mod buckets], 32-bit; a sequence's first token takes
+    the row `buckets` of `pairs` [buckets + 1, dim]. The previous token is state of the request: one number in a slot, a cache
+    layer of its own that the model numbers behind those of the blocks."""
+
+    def __init__(self, vocab: int, dim: int, buckets: int, mul_prev: int, mul_cur: int, names: Dict[str, str]):
+        super().__init__(names)
+        self.vocab, self.dim, self.buckets, self.mul_prev, self.mul_cur = vocab, dim, int(buckets), int(mul_prev), int(mul_cur)
+        self.table = self.pairs = None
+
+    def local_specs(self):
+        return {"table": TensorSpec((self.vocab, self.dim), MATRIX), "pairs": TensorSpec((self.buckets + 1, self.dim), MATRIX)}
+
+    def cache_spec(self):
+        return StateSpec((1,), "int32")
+
+    def forward(self, ctx, out: Optional[torch.Tensor] = None, cache_layer: Optional[int] = None) -> torch.Tensor:
+        x = ctx.empty((ctx.T, self.dim), torch.float32) if out is None else out
+        ops.embed_pairs(self.table, self.pairs, ctx.token_ids, ctx.positions, ctx.tok_req, ctx.cu_q, ctx.slots, ctx.state(cache_layer),
+                        self.mul_prev, self.mul_cur, x)
         return x
 
 

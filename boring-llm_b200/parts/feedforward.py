@@ -283,14 +283,21 @@ class RoutedExperts(FeedForward):
     itself, the weights are the softmax over the chosen logits alone); `router_bias`: z = h Wr^T + b; `group_score` "top2" (the sum
     of a group's two largest choice scores) or "max" (its largest); `n_identity`: the router has `n_experts + n_identity`
     outputs, and the last `n_identity` are identity experts without tensors whose output is the input row h itself (times
-    the weight); groups are formed over experts and identity experts together."""
+    the weight); groups are formed over experts and identity experts together; `weight_on` "output" (the result is the sum of
+    w * expert(h)) or "input" (the sum of expert(w * h): the weight multiplies what the expert reads).
+
+    `apply_pairs` leaves the sum over a token's experts to the caller (a kernel that passes over the rows anyway)."""
     graph_safe = True
     SCORES = {"sigmoid": ops.SCORE_SIGMOID, "softmax": ops.SCORE_SOFTMAX, "chosen": ops.SCORE_CHOSEN}
 
     def __init__(self, dim: int, hidden: int, n_experts: int, top: int, names: Dict[str, str], n_groups: int = 1,
                  keep_groups: int = 1, correction: bool = True, activation: str = "silu", limit: float = 0.0,
-                 score: str = "sigmoid", group_score: str = "top2", n_identity: int = 0, router_bias: bool = False):
+                 score: str = "sigmoid", group_score: str = "top2", n_identity: int = 0, router_bias: bool = False,
+                 weight_on: str = "output"):
         super().__init__(names)
+        if weight_on not in ("output", "input") or (weight_on == "input" and n_identity):
+            raise ValueError(f"RoutedExperts: weight_on {weight_on!r} with {n_identity} identity experts")
+        self.weight_input = weight_on == "input"
         self.has_router_bias, self.b_router = bool(router_bias), None
         if score not in self.SCORES or group_score not in ("top2", "max") or n_identity < 0:
             raise ValueError(f"RoutedExperts: score {score!r}, group_score {group_score!r}, {n_identity} identity experts")
@@ -367,28 +374,47 @@ class RoutedExperts(FeedForward):
             self.record.append(ids.clone())
         return ids, wts
 
-    def _run(self, ctx, h, out, add):
+    def _pairs(self, ctx, h):
+        """The experts' results, one 32-bit row for every (token, chosen expert): (rows, the row of each pair or None for the
+        pairs' own order, the weights their sum takes or None for ones, the choice)."""
         T = h.shape[0]
         ids, wts = self.route(ctx, h)
+        scale, left = (wts, None) if self.weight_input else (None, wts)
         if ctx.fast and ops.grouped_gemm_supported(h, self.w_gate_up) and self.hidden % 8 == 0:
             # tensor cores: the pairs lie expert by expert in tiles of 128 rows, each tile multiplied by its expert's matrices
             pos, row_src, tile_expert = ops.moe_plan(ids, self.E)
             rows = ctx.empty((row_src.numel(), self.dim))
-            ops.gather_rows(h, row_src, self.top, rows)
+            ops.gather_rows(h, row_src, self.top, rows, scale)
             act = ctx.empty((row_src.numel(), self.hidden))
             ops.gemm_grouped(rows, self.w_gate_up, tile_expert, act, EPI_SWIGLU, self.act_args)
             y = ctx.empty((row_src.numel(), self.dim), torch.float32)
             ops.gemm_grouped(act, self.w_down, tile_expert, y, EPI_NONE)
-            ops.moe_combine_rows(y, pos, wts, out, add=add, x=h if self.n_identity else None)
-            return
+            return y, pos, left, ids
+        rows, per = h, self.top
+        if scale is not None:
+            rows, per = ctx.empty((T * self.top, self.dim)), 1
+            ops.scale_pairs(h, scale, rows)
         act = ctx.empty((T * self.top, self.hidden))
-        ops.expert_gemm_plain(h, self.top, self.w_gate_up, ids, act, EPI_SWIGLU, self.act_args)
+        ops.expert_gemm_plain(rows, per, self.w_gate_up, ids, act, EPI_SWIGLU, self.act_args)
         y = ctx.empty((T * self.top, self.dim), torch.float32)
         ops.expert_gemm_plain(act, 1, self.w_down, ids, y, EPI_NONE)
-        if self.n_identity:
+        return y, None, left, ids
+
+    def _run(self, ctx, h, out, add):
+        y, pos, wts, ids = self._pairs(ctx, h)
+        if pos is not None:
+            ops.moe_combine_rows(y, pos, wts, out, add=add, x=h if self.n_identity else None)
+        elif self.n_identity:
             ops.moe_combine(y, wts, out, add=add, ids=ids, n_real=self.E, x=h)
         else:
-            ops.moe_combine(y, wts, out, add=add)
+            ops.moe_combine(y, wts, out, add=add, top=self.top)
+
+    def apply_pairs(self, ctx, h):
+        """(rows, row of each pair or None, weights or None): token t's result is the sum over k < top of weights[t, k] (None: 1)
+        times rows[pos[t * top + k]] (None: row t * top + k). None: the caller uses `apply` (identity experts)."""
+        if self.n_identity:
+            return None
+        return self._pairs(ctx, h)[:3]
 
     def forward(self, ctx, h, residual):
         self._run(ctx, h, residual, True)

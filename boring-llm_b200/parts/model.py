@@ -38,12 +38,15 @@ class DecoderModel(Part):
 
     def __init__(self, embedding, blocks: Sequence[Part], final_norm, head,
                  schedule: Optional[Sequence[LayerCall]] = None, ignorable_tensors: Sequence[str] = (),
-                 depth_mix: Optional[Sequence[Part]] = None, reentry: Optional[Part] = None):
+                 depth_mix: Optional[Sequence[Part]] = None, reentry: Optional[Part] = None, streams: int = 0):
         """`reentry`: the part (`parts.depth.StreamReentry`) that runs ahead of every entry of the run order with `enters`.
         `depth_mix`: one part per entry of the run order (`parts.depth.DepthWeightedAverage`); entry i's part turns the
         streams X_0 .. X_(i+1) (the embedding rows and what each entry so far left) into what the next entry, or the
-        final norm, reads. Without it every entry reads what the one before left."""
+        final norm, reads. Without it every entry reads what the one before left. `streams` n > 0: the residual is n streams
+        that start as the embedding rows, the blocks (`HyperBlock`) work on all of them, and the final norm reads their sum. An
+        embedding that keeps state (its `cache_spec()`) gets a cache layer behind those of the run order."""
         super().__init__()
+        self.streams = int(streams)
         self.embedding, self.blocks, self.final_norm, self.head = embedding, list(blocks), final_norm, head
         self.depth_mix = list(depth_mix) if depth_mix is not None else None
         self.reentry = reentry
@@ -63,6 +66,10 @@ class DecoderModel(Part):
                     raise ValueError(f"an entry reads cache layer {c} before any entry writes it")
         if any(call.enters for call in self.schedule) and (reentry is None or self.depth_mix is not None):
             raise ValueError("entries of the run order that begin a pass need a `reentry` part (and no depth mix)")
+        if self.streams and (reentry is not None or self.depth_mix is not None):
+            raise ValueError("a residual of several streams does not go with a reentry or a depth mix")
+        spec = getattr(embedding, "cache_spec", None)
+        self.embedding_cache = 1 + max(written, default=-1) if spec is not None and spec() is not None else None
         if self.depth_mix is not None and len(self.depth_mix) != len(self.schedule):
             raise ValueError(f"{len(self.depth_mix)} depth-mix parts for {len(self.schedule)} entries of the run order")
 
@@ -113,7 +120,14 @@ class DecoderModel(Part):
                 if specs[c] is not None and specs[c] != sp:
                     raise ValueError(f"cache layer {c} is shared by layers with different needs")
                 specs[c] = sp
+        if self.embedding_cache is not None:
+            specs.append(self.embedding.cache_spec())
         return specs
+
+    def _embed(self, ctx, out=None) -> torch.Tensor:
+        if self.embedding_cache is not None:
+            return self.embedding.forward(ctx, out, self.embedding_cache)
+        return self.embedding.forward(ctx, out=out)
 
     def forward(self, ctx) -> torch.Tensor:
         """Runs the tokens of `ctx` through every layer and returns 32-bit logits at `ctx.logit_rows`."""
@@ -121,7 +135,9 @@ class DecoderModel(Part):
         if self.depth_mix is not None:
             x = self._forward_depth_mixed(ctx)
             return self._logits(ctx, x)
-        x = x0 = self.embedding.forward(ctx)
+        if self.streams:
+            return self._forward_streams(ctx)
+        x = x0 = self._embed(ctx)
         if self.reentry is not None and not self.schedule[0].enters:
             x = x0.clone()                      # blocks add into the stream in place; the embedding rows are read again
         for i, call in enumerate(self.schedule):
@@ -144,7 +160,7 @@ class DecoderModel(Part):
         writes stream i + 2. Nothing is copied but the embedding rows, once."""
         n = len(self.schedule)
         streams = ctx.empty((n + 2, ctx.T, self.embedding.dim), torch.float32)
-        self.embedding.forward(ctx, out=streams[0])
+        self._embed(ctx, streams[0])
         streams[1].copy_(streams[0])
         ctx.norm_after_block = None
         from .depth import AfterBlock
@@ -157,6 +173,18 @@ class DecoderModel(Part):
             after.run_unfused(ctx)
         ctx.memo["streams"] = streams            # for whoever wants to look at the stream after each entry (tests)
         return streams[n + 1]
+
+    def _forward_streams(self, ctx) -> torch.Tensor:
+        from .streams import StreamResidual
+        ctx.norm_after_block = None
+        streams = StreamResidual(self._embed(ctx), self.streams)
+        for call in self.schedule:
+            self.blocks[call.block].forward(ctx, streams, call.cache, call.write_cache)
+            if self.keep_streams is not None:
+                self.keep_streams.append(streams.total(ctx))
+        if ctx.logit_rows.shape[0] == 0:
+            return ctx.empty((0, self.vocab_size), torch.float32)
+        return self.head.forward(ctx, streams.final(ctx, self.final_norm, ctx.logit_rows))
 
     def _logits(self, ctx, x) -> torch.Tensor:
         if ctx.logit_rows.shape[0] == 0:

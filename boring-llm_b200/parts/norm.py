@@ -15,10 +15,13 @@ class RMSNorm(Part):
     (src/math.br:18-36). Input: the 32-bit residual stream; output: the engine's activation dtype.
     `scalar_weight`: the checkpoint holds ONE number (a tensor without dimensions) that multiplies every coordinate; it is
     spread over the width when it is placed, so every kernel that takes an RMS norm's weight takes this one.
-    `around_zero`: the checkpoint holds w - 1; the weight 1 + w is formed in 32-bit when it is placed."""
+    `around_zero`: the checkpoint holds w - 1; the weight 1 + w is formed in 32-bit when it is placed. `gain`: a constant on
+    the normed rows, multiplied into the weight in 32-bit when it is placed (a factor on the logits behind a final norm)."""
 
-    def __init__(self, dim: int, eps: float, names: Dict[str, str], scalar_weight: bool = False, around_zero: bool = False):
+    def __init__(self, dim: int, eps: float, names: Dict[str, str], scalar_weight: bool = False, around_zero: bool = False,
+                 gain: float = 1.0):
         super().__init__(names)
+        self.gain = float(gain)
         self.dim, self.eps, self.scalar_weight, self.around_zero = dim, float(eps), bool(scalar_weight), bool(around_zero)
         self.weight: Optional[torch.Tensor] = None
 
@@ -31,6 +34,8 @@ class RMSNorm(Part):
             w = w.reshape(1).expand(self.dim).contiguous()
         if self.around_zero:
             w = w.to(torch.float32) + 1.0
+        if self.gain != 1.0:
+            w = w.to(torch.float32) * self.gain
         self.weight = to_device_vector(w, dtype, device)
 
     def forward(self, ctx, x: torch.Tensor, row_idx: Optional[torch.Tensor] = None, pending_ok: bool = False):

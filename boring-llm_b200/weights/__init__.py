@@ -1,6 +1,6 @@
 from .safetensors_io import SafetensorsError, SafetensorsFile, write_safetensors, open_model_files
 from .loader import (TensorSpec, WeightsError, load_checkpoint, write_model_folder,
-                     MATRIX, NORM, BIAS, INT_TABLE)
+                     MATRIX, NORM, BIAS, INT_TABLE, MIXING)
 from .random_init import RandomTensors, random_tensor, tensor_key
 
 
@@ -14,5 +14,5 @@ def random_tensors(expected, seed, dtype=None, std=0.02, vocab_size=0, device="c
 __all__ = [
     "SafetensorsError", "SafetensorsFile", "write_safetensors", "open_model_files", "TensorSpec",
     "WeightsError", "load_checkpoint", "random_tensors", "random_tensor", "tensor_key", "RandomTensors",
-    "write_model_folder", "MATRIX", "NORM", "BIAS", "INT_TABLE",
+    "write_model_folder", "MATRIX", "NORM", "BIAS", "INT_TABLE", "MIXING",
 ]

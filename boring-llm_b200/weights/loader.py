@@ -17,7 +17,7 @@ import torch
 from .safetensors_io import SafetensorsError, open_model_files, write_safetensors
 
 # what a tensor is, which decides how the random-weights mode fills it
-MATRIX, NORM, BIAS, INT_TABLE = "matrix", "norm", "bias", "int_table"
+MATRIX, NORM, BIAS, INT_TABLE, MIXING = "matrix", "norm", "bias", "int_table", "mixing"
 
 
 @dataclass(frozen=True)
@@ -25,7 +25,7 @@ class TensorSpec:
     """`shape`: a dimension of -1 is a size that only the checkpoint gives (the inner size of a product in two
     factors); the part that owns the tensor reads it when the tensor is placed."""
     shape: Tuple[int, ...]
-    kind: str = MATRIX          # MATRIX | NORM | BIAS | INT_TABLE
+    kind: str = MATRIX          # MATRIX | NORM | BIAS | INT_TABLE | MIXING (a small square matrix around the identity)
     high: int = 0               # INT_TABLE: the values lie in [0, high) and differ within a row (0: token ids, any)
 
 

@@ -37,7 +37,7 @@ from typing import Dict, Iterator
 
 import torch
 
-from .loader import BIAS, INT_TABLE, MATRIX, NORM, TensorSpec
+from .loader import BIAS, INT_TABLE, MATRIX, MIXING, NORM, TensorSpec
 
 _M64 = (1 << 64) - 1
 _STEP = 0x9E3779B97F4A7C15
@@ -118,7 +118,8 @@ def _normal_chunk(key: int, start: int, n: int, device) -> torch.Tensor:
 
 def random_tensor(name: str, spec: TensorSpec, seed: int, dtype: torch.dtype = torch.bfloat16, std: float = 0.02,
                   vocab_size: int = 0, device="cpu") -> torch.Tensor:
-    """The tensor `name` of the random model `seed`: matrices and biases N(0, std), norm weights 1 + N(0, std),
+    """The tensor `name` of the random model `seed`: matrices and biases N(0, std), norm weights 1 + N(0, std), mixing matrices
+    the identity plus N(0, std),
     integer tables uniform in [0, vocab_size), stored as `dtype` (integer tables as int32)."""
     device = torch.device(device)
     if any(int(d) < 0 for d in spec.shape):
@@ -147,6 +148,9 @@ def random_tensor(name: str, spec: TensorSpec, seed: int, dtype: torch.dtype = t
         v = _normal_chunk(key, start, m, device) * float(std)
         if spec.kind == NORM:
             v = v + 1.0
+        elif spec.kind == MIXING:                   # the identity plus noise: [n, n], element i on the diagonal where i mod (n + 1) = 0
+            at = torch.arange(start, start + m, device=device)
+            v = v + (at % (int(spec.shape[-1]) + 1) == 0).to(torch.float64)
         elif spec.kind not in (MATRIX, BIAS):
             raise ValueError(f"tensor {name}: unknown kind {spec.kind!r}")
         out[start:start + m] = v.to(torch.float32).to(dtype)
