@@ -10,6 +10,7 @@ its roofline.
     python bench.py --design miforax [--sizes 0.5b|3b] [--layers L]     # the Miforax design beside Fezopel and Qwen2 at equal sizes
     python bench.py --design dapuzen [--sizes 0.5b|3b] [--layers L]     # the Dapuzen design beside Fezopel and Qwen2 at equal sizes
     python bench.py --design gipinex [--sizes 0.5b|3b] [--layers L]     # the Gipinex design beside Miforax and Kavotar at equal sizes
+    python bench.py --design zuvevik [--sizes 0.5b|3b] [--layers L]     # the Zuvevik design beside Fezopel and Kavotar at equal sizes
 
 One JSON line on standard output. A "step" is one decode step of the whole batch. Requests are real ones: random
 prompts admitted by the scheduler, prefilled in portions through the engine, then decoded; the model comes from the
@@ -490,6 +491,27 @@ def gipinex_config(sizes, n_layers):
                                       "max_position_embeddings": 32768})
 
 
+ZUVEVIK_STREAMS, ZUVEVIK_WINDOW, ZUVEVIK_BUCKETS = 4, 1024, 65521
+ZUVEVIK_EXPERTS, ZUVEVIK_TOP = KAVOTAR_EXPERTS, KAVOTAR_TOP
+
+
+def zuvevik_config(sizes, n_layers):
+    """A Zuvevik model with the width, heads, head size, layers and vocabulary of a Qwen2.5 size: four streams, Fezopel's window of
+    1,024 in every layer, all layers blend their values; the first layer has the dense feed-forward, the others Kavotar's 16
+    experts of a quarter of its hidden size, 4 a token."""
+    import boring_llm_b200 as b
+    s = SIZES[sizes]
+    d, H, KV, dh, F, V = (s[k] for k in ("hidden_size", "num_attention_heads", "num_key_value_heads", "head_dim",
+                                         "intermediate_size", "vocab_size"))
+    mixer = {"heads": H, "kv_heads": KV, "dim": dh, "vdim": dh, "mask": {"size": ZUVEVIK_WINDOW}, "rot": {"base": 1000000.0, "dims": dh},
+             "scale": dh ** -0.5, "v_mix": True}
+    moe = {"kind": "moe", "expert": {"ff": F // ZUVEVIK_TOP // 8 * 8, "limit": 7.0}, "router": {"experts": ZUVEVIK_EXPERTS, "top": ZUVEVIK_TOP}}
+    layers = [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": F} if i == 0 else moe} for i in range(n_layers)]
+    return b.ZuvevikConfig.from_dict({"architecture": "Zuvevik", "vocab": V, "width": d, "norm": {"eps": 1e-6}, "streams": ZUVEVIK_STREAMS,
+                                      "logit_scale": 0.5, "embedding": {"bigram": {"buckets": ZUVEVIK_BUCKETS, "mul_prev": 31337, "mul_cur": 271}},
+                                      "layers": layers, "max_position_embeddings": 32768})
+
+
 def kernel_time_line(eng, entries, again):
     """The time of every kernel of one step INSIDE its captured graph: the step is captured with a time stamp between
     every two kernels, then `again` (the same shape: it replays that graph) runs, and the stamps of the replay give
@@ -533,8 +555,9 @@ def design_bench(args):
     pk = peaks()
     n_layers = args.layers or 8
     makers = {"fezopel": fezopel_config, "kavotar": kavotar_config, "miforax": miforax_config, "dapuzen": dapuzen_config,
-              "gipinex": gipinex_config, "qwen2": lambda sizes, n: b.Qwen2Config.from_dict({**COMMON, **SIZES[sizes], "num_hidden_layers": n})}
-    names = {"fezopel": ("fezopel", "qwen2"), "gipinex": ("gipinex", "miforax", "kavotar")}.get(args.design, (args.design, "fezopel", "qwen2"))
+              "gipinex": gipinex_config, "zuvevik": zuvevik_config, "qwen2": lambda sizes, n: b.Qwen2Config.from_dict({**COMMON, **SIZES[sizes], "num_hidden_layers": n})}
+    names = {"fezopel": ("fezopel", "qwen2"), "gipinex": ("gipinex", "miforax", "kavotar"),
+             "zuvevik": ("zuvevik", "fezopel", "kavotar")}.get(args.design, (args.design, "fezopel", "qwen2"))
     out = {"design": args.design, "beside": list(names[1:]), "sizes": args.sizes, "layers": n_layers, "dtype": "bf16", "data": "synthetic",
            "context": CONTEXT, "prefill_tokens": PREFILL_TOKENS, "peaks": pk["source"], "models": {}}
     if args.design == "fezopel":
@@ -547,6 +570,8 @@ def design_bench(args):
     elif args.design == "gipinex":
         out.update(pattern=list(GIPINEX_PATTERN), loop=[0, GIPINEX_LOOP, 2], experts=[MIFORAX_EXPERTS, MIFORAX_TOP],
                    latent=list(MIFORAX_LATENT[args.sizes]))
+    elif args.design == "zuvevik":
+        out.update(streams=ZUVEVIK_STREAMS, window=ZUVEVIK_WINDOW, experts=[ZUVEVIK_EXPERTS, ZUVEVIK_TOP])
     else:
         out.update(pattern=list(KAVOTAR_PATTERN), chunk=KAVOTAR_CHUNK, experts=[KAVOTAR_EXPERTS, KAVOTAR_TOP, KAVOTAR_GROUPS, KAVOTAR_KEEP])
     clocks = ClockSampler()
@@ -612,7 +637,7 @@ def main():
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "prefill4", "mixed"],
                     help="run one part only and print its figures (for profilers; not the benchmark line)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--design", default="", choices=["", "fezopel", "kavotar", "miforax", "dapuzen", "gipinex"],
+    ap.add_argument("--design", default="", choices=["", "fezopel", "kavotar", "miforax", "dapuzen", "gipinex", "zuvevik"],
                     help="measure another design beside its closest models at equal sizes instead of the default workload (its own JSON line)")
     args = ap.parse_args()
     if args.impl == "reference":

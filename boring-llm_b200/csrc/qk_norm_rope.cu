@@ -13,7 +13,8 @@ constexpr int THREADS = 128;
 // Further options. norm_q / norm_k > 0: how many of a row's values the whole-row norms average over (heads that are padded
 // with zeros count their own values only). first: values of the same tokens that another layer projected, blended into this
 // layer's ones: heads of first_dv values, first_places apart; this layer's heads have dv values of their own (then zeros).
-struct BlBlendArgs { int norm_q, norm_k; const float* first; int ld_first, first_dv, first_places, dv; const void* lambda; int lambda_dtype; };
+// same: both rows are laid out alike and the other one lies in 16-byte pieces.
+struct BlBlendArgs { int norm_q, norm_k; const float* first; int ld_first, first_dv, first_places, dv; const void* lambda; int lambda_dtype; int same; };
 
 __device__ __forceinline__ float block_sum(float v, float* part) {
     v = bl_warp_sum(v);
@@ -115,6 +116,140 @@ qk_norm_rope_write_kernel(const float* proj, int ld, int off_k, int off_v, const
     }
 }
 
+// The same four values at a time, for rows, heads and rotated parts that are multiples of four and rotation in halves: the
+// token's q and k rows are read once, into shared memory, with both sums of squares on the way; positions, angles and page
+// numbers are worked out before the kernel's predecessor has finished.
+constexpr int FAST_THREADS = 512;
+
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a), *reinterpret_cast<const unsigned*>(&b));
+}
+__device__ __forceinline__ float4 weights4(const void* w, int dtype, int i) {
+    if (!w) return make_float4(1.f, 1.f, 1.f, 1.f);
+    if (dtype == BL_F32) return *reinterpret_cast<const float4*>((const float*)w + i);
+    const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)w + i);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename TT>
+__global__ void __launch_bounds__(FAST_THREADS)
+qk_norm_rope_write4_kernel(const float* proj, int ld, int off_k, int off_v, const void* __restrict__ qw, int qw_dtype,
+                           const void* __restrict__ kw, int kw_dtype, float eps, const int* __restrict__ positions,
+                           const int* __restrict__ tok_req, const int* __restrict__ block_table, int max_pages,
+                           const float* __restrict__ inv_freq, int rot_half, TT* __restrict__ q_out,
+                           TT* __restrict__ k_cache, TT* __restrict__ v_cache, int H, int KV, int dk, int dv, int page_size,
+                           int per_head, const float* __restrict__ q_head_scale, BlBlendArgs bl) {
+    bl_pdl_trigger();
+    extern __shared__ __align__(16) float sm4[];       // cos, sin [rot_half] each, the q and k rows [(H + KV) * dk], 1 / rms per head
+    __shared__ float part[2][FAST_THREADS / 32];
+    const int t = blockIdx.x, nq = H * dk, nk = KV * dk;
+    float* cs = sm4;
+    float* sn = cs + rot_half;
+    float* x = sn + rot_half;
+    float* inv_head = x + nq + nk;
+    const int pos = positions[t], r = tok_req[t];
+    for (int j = threadIdx.x; j < rot_half; j += blockDim.x) {
+        const float a = (float)pos * inv_freq[j];
+        cs[j] = cosf(a);
+        sn[j] = sinf(a);
+    }
+    const int page = k_cache || v_cache ? block_table[(size_t)r * max_pages + pos / page_size] : 0;
+    const int in_page = pos % page_size;
+    const float lam = bl.first ? bl_load_any(bl.lambda, bl.lambda_dtype, 0) : 0.f;
+    bl_pdl_wait();
+    const float* row = proj + (size_t)t * ld;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x * 4; i < nq + nk; i += blockDim.x * 4) {
+        const float4 f = *reinterpret_cast<const float4*>(row + (i < nq ? i : off_k + i - nq));
+        *reinterpret_cast<float4*>(x + i) = f;
+        const float s = (f.x * f.x + f.y * f.y) + (f.z * f.z + f.w * f.w);
+        if (i < nq) sq += s; else sk += s;
+    }
+    if (v_cache) {                                     // (no norm, no rotation: they need not wait for the sums)
+        for (int e = threadIdx.x * 4; e < KV * dv; e += blockDim.x * 4) {
+            const int g = e / dv, d = e % dv;
+            const float4 f = *reinterpret_cast<const float4*>(row + off_v + e);
+            float v[4] = {f.x, f.y, f.z, f.w};
+            if (bl.first && bl.same) {
+                const float4 o = *reinterpret_cast<const float4*>(bl.first + (size_t)t * bl.ld_first + e);
+                v[0] = (1.f - lam) * v[0] + lam * o.x;
+                v[1] = (1.f - lam) * v[1] + lam * o.y;
+                v[2] = (1.f - lam) * v[2] + lam * o.z;
+                v[3] = (1.f - lam) * v[3] + lam * o.w;
+            } else if (bl.first) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    float o = 0.f;
+                    if (d + j < bl.dv) {
+                        const int flat = g * bl.dv + d + j;
+                        o = bl.first[(size_t)t * bl.ld_first + (flat / bl.first_dv) * bl.first_places + flat % bl.first_dv];
+                    }
+                    v[j] = (1.f - lam) * v[j] + lam * o;
+                }
+            }
+            store4(v_cache + (((size_t)page * KV + g) * page_size + in_page) * dv + d, v);
+        }
+    }
+    float inv_q = 1.f, inv_k = 1.f;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    if (!per_head) {
+        sq = bl_warp_sum(sq);
+        sk = bl_warp_sum(sk);
+        if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
+    }
+    __syncthreads();
+    if (per_head) {
+        for (int hh = warp; hh < H + KV; hh += warps) {
+            float s = 0.f;
+            for (int i = lane; i < dk; i += 32) s += x[hh * dk + i] * x[hh * dk + i];
+            s = bl_warp_sum(s);
+            if (lane == 0) inv_head[hh] = ((hh < H ? qw : kw) != nullptr) ? 1.0f / sqrtf(s / (float)dk + eps) : 1.f;
+        }
+        __syncthreads();
+    } else {
+        float a = 0.f, b = 0.f;
+        for (int i = 0; i < warps; ++i) { a += part[0][i]; b += part[1][i]; }
+        if (qw) inv_q = 1.0f / sqrtf(a / (float)(bl.norm_q > 0 ? bl.norm_q : nq) + eps);
+        if (kw) inv_k = 1.0f / sqrtf(b / (float)(bl.norm_k > 0 ? bl.norm_k : nk) + eps);
+    }
+    for (int e = threadIdx.x * 4; e < nq + nk; e += blockDim.x * 4) {
+        const bool is_q = e < nq;
+        const int hh = e / dk, d = e - hh * dk;
+        const int wbase = per_head ? 0 : (is_q ? hh * dk : (hh - H) * dk);
+        const void* w = is_q ? qw : kw;
+        const int wd = is_q ? qw_dtype : kw_dtype;
+        const float inv = per_head ? inv_head[hh] : (is_q ? inv_q : inv_k);
+        const float4 m = *reinterpret_cast<const float4*>(x + e);
+        const float4 mw = weights4(w, wd, wbase + d);
+        float v[4] = {m.x * inv * mw.x, m.y * inv * mw.y, m.z * inv * mw.z, m.w * inv * mw.w};
+        if (d < 2 * rot_half) {
+            const bool first = d < rot_half;
+            const int od = first ? d + rot_half : d - rot_half, j = first ? d : d - rot_half;
+            const float4 o = *reinterpret_cast<const float4*>(x + hh * dk + od);
+            const float4 ow = weights4(w, wd, wbase + od);
+            const float4 c = *reinterpret_cast<const float4*>(cs + j), s4 = *reinterpret_cast<const float4*>(sn + j);
+            const float sg = first ? -1.f : 1.f;
+            v[0] = v[0] * c.x + sg * (o.x * inv * ow.x) * s4.x;
+            v[1] = v[1] * c.y + sg * (o.y * inv * ow.y) * s4.y;
+            v[2] = v[2] * c.z + sg * (o.z * inv * ow.z) * s4.z;
+            v[3] = v[3] * c.w + sg * (o.w * inv * ow.w) * s4.w;
+        }
+        if (is_q) {
+            if (q_head_scale) {
+                const float f = q_head_scale[hh];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) v[j] *= f;
+            }
+            store4(q_out + (size_t)t * nq + e, v);
+        } else if (k_cache) {
+            store4(k_cache + (((size_t)page * KV + (hh - H)) * page_size + in_page) * dk + d, v);
+        }
+    }
+}
+
 }  // namespace
 
 extern "C" int bl_qk_norm_rope_write(const float* proj, int ld, int off_k, int off_v, const void* q_norm_w, int qw_dtype,
@@ -154,8 +289,27 @@ extern "C" int bl_qk_norm_rope_write_ext(const float* proj, int ld, int off_k, i
     if (v_first && (!lambda || dv_real <= 0 || dv_real > dv || first_dv <= 0 || first_dv > first_places || KV * dv_real % first_dv != 0 ||
                     ld_first < KV * dv_real / first_dv * first_places))
         BL_FAIL("bl_qk_norm_rope_write: values of %d heads of %d cannot be blended with heads of %d in rows of %d", KV, dv_real, first_dv, ld_first);
-    const BlBlendArgs bl{norm_q, norm_k, v_first, ld_first, first_dv, first_places, dv_real, lambda, lambda_dtype};
+    const int same = v_first && first_dv == dv_real && first_places == dv && ld_first % 4 == 0 && ((uintptr_t)v_first & 15) == 0;
+    const BlBlendArgs bl{norm_q, norm_k, v_first, ld_first, first_dv, first_places, dv_real, lambda, lambda_dtype, same};
     cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem4 = (size_t)(2 * rot_half + (H + KV) * dk + (per_head ? H + KV : 0)) * sizeof(float);
+    const bool fours = (pair_layout == BL_PAIRS_HALVES || rot_half == 0) && dk % 4 == 0 && dv % 4 == 0 && rot_half % 4 == 0 && ld % 4 == 0 &&
+                       off_k % 4 == 0 && off_v % 4 == 0 && smem4 <= 48 * 1024 &&
+                       (((uintptr_t)proj | (uintptr_t)q_norm_w | (uintptr_t)k_norm_w | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
+    if (fours) {
+        int threads = ((H + KV) * dk / 4 + 31) / 32 * 32;
+        const int most = T <= 256 ? FAST_THREADS : 256;
+        if (threads > most) threads = most;
+#define BL_GO(TT) BL_CUDA(bl_launch_dependent(qk_norm_rope_write4_kernel<TT>, dim3(T), dim3(threads), smem4, s, proj, ld, off_k, off_v, \
+        q_norm_w, qw_dtype, k_norm_w, kw_dtype, eps, positions, tok_req, block_table, max_pages, inv_freq, rot_half, \
+        (TT*)q_out, (TT*)k_cache, (TT*)v_cache, H, KV, dk, dv, page_size, per_head, q_head_scale, bl))
+        if (dtype == BL_F32) BL_GO(float);
+        else if (dtype == BL_BF16) BL_GO(__nv_bfloat16);
+        else BL_FAIL("bl_qk_norm_rope_write: unknown dtype %d", dtype);
+#undef BL_GO
+        BL_CHECK_LAUNCH("bl_qk_norm_rope_write");
+        return 0;
+    }
     const size_t smem = (size_t)(2 * rot_half + 1 + (per_head ? H + KV : 0)) * sizeof(float);
 #define BL_GO(TT) BL_CUDA(bl_launch_dependent(qk_norm_rope_write_kernel<TT>, dim3(T), dim3(THREADS), smem, s, proj, ld, off_k, off_v, \
         q_norm_w, qw_dtype, k_norm_w, kw_dtype, eps, positions, tok_req, block_table, max_pages, inv_freq, rot_half, pair_layout, \
