@@ -11,7 +11,7 @@
 namespace {
 
 constexpr int MAX_STREAMS = 16;
-constexpr int MAX_THREADS = 256;
+constexpr int MAX_THREADS = 512;
 
 template <int VEC> struct Lane;
 template <> struct Lane<4> {
@@ -43,7 +43,7 @@ struct HyperArgs {
 
 // S > 0: that many streams; S = 0: `n`, up to MAX_STREAMS.
 template <int S, int VEC, typename TH>
-__global__ void __launch_bounds__(MAX_THREADS)
+__global__ void __launch_bounds__(S == 0 ? 256 : MAX_THREADS, S >= 1 && S <= 4 ? 2 : 1)
 hyper_step_kernel(const HyperArgs p) {
     bl_pdl_trigger();
     constexpr int NS = S > 0 ? S : MAX_STREAMS;
@@ -66,6 +66,7 @@ hyper_step_kernel(const HyperArgs p) {
     const float* y0 = nullptr;
     if (p.write && !p.y_pos && p.top == 1 && !p.y_wts) y0 = p.y + t * p.d;
     float ss = 0.f;
+#pragma unroll 1
     for (int c = threadIdx.x * VEC; c < p.d; c += blockDim.x * VEC) {
         Lane<VEC> x[NS], y;
         if (p.x_stride == 0) {
@@ -159,7 +160,8 @@ hyper_step_kernel(const HyperArgs p) {
 template <int S, int VEC>
 int launch_hyper(const HyperArgs& a, int rows, cudaStream_t s) {
     int threads = ((a.d + VEC - 1) / VEC + 31) / 32 * 32;
-    if (threads > MAX_THREADS) threads = MAX_THREADS;
+    const int most = S > 0 && rows <= 256 ? MAX_THREADS : 256;                 // few rows: a step waits for one row's way through
+    if (threads > most) threads = most;
     const size_t smem = (size_t)(2 * MAX_STREAMS + MAX_STREAMS * MAX_STREAMS + a.d) * sizeof(float);
     if (smem > 200 * 1024) BL_FAIL("bl_hyper_step: rows of %d values do not fit shared memory", a.d);
     if (a.h_dtype == BL_BF16) {
@@ -180,6 +182,10 @@ int dispatch_hyper(const HyperArgs& a, int rows, cudaStream_t s) {
         case 2: return launch_hyper<2, VEC>(a, rows, s);
         case 3: return launch_hyper<3, VEC>(a, rows, s);
         case 4: return launch_hyper<4, VEC>(a, rows, s);
+        case 5: return launch_hyper<5, VEC>(a, rows, s);
+        case 6: return launch_hyper<6, VEC>(a, rows, s);
+        case 7: return launch_hyper<7, VEC>(a, rows, s);
+        case 8: return launch_hyper<8, VEC>(a, rows, s);
         default: return launch_hyper<0, VEC>(a, rows, s);
     }
 }
