@@ -127,7 +127,7 @@ class DecoderModel(Part):
     def _embed(self, ctx, out=None) -> torch.Tensor:
         if self.embedding_cache is not None:
             return self.embedding.forward(ctx, out, self.embedding_cache)
-        return self.embedding.forward(ctx, out=out)
+        return self.embedding.forward(ctx) if out is None else self.embedding.forward(ctx, out=out)
 
     def forward(self, ctx) -> torch.Tensor:
         """Runs the tokens of `ctx` through every layer and returns 32-bit logits at `ctx.logit_rows`."""
